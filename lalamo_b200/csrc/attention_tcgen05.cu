@@ -342,9 +342,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const bool needs_mask = key0 + kTaKeys - 1 > first_position || (p.window > 0 && key0 < last_position - p.window + 1);
             // The row is read twice, 32 scores at a time (once for its maximum, once for its terms): a
             // thread then needs half the registers, and three CTAs fit an SM.  Both passes exist with and
-            // without the mask, chosen by one branch per tile: with the test inside the loops the
-            // compiler evaluated the mask's comparisons for every score of every tile (four ALU
-            // instructions per score and pass, which made the ALU pipe the kernel's limit).
+            // without the mask, chosen by one branch per tile: with the test inside the loops the mask's
+            // comparisons ran for every score of every tile, and the ALU pipe was the kernel's limit.
             float tops[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             auto row_maximum = [&](auto masked) {
                 constexpr bool kMasked = decltype(masked)::value;
