@@ -10,6 +10,8 @@ rule, and slots for per-request state of fixed size.
 * Pages are given back when a request ends, and, in a windowed group, as soon as the window has
   passed them (the pages of the kept first positions stay); they are handed out again (last freed
   first) without being cleared.
+* A need may borrow the keys and values of the entry that ``cache_from`` names beside cells of its own
+  (:class:`BorrowedKVNeed`); the pages then stay for as long as the owner or any borrower may look at them.
 * A mixer may declare several needs at once (:class:`CompositeNeed`, nested at will): the manager
   treats every leaf as a *cell* of its own and hands the mixer a :class:`CompositeView` of the same
   shape.  A schedule entry with a plain need is one cell.
@@ -25,12 +27,12 @@ The reference has no counterpart: it holds one contiguous cache per sequence
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 
 import torch
 
 from .. import ops
-from ..parts.base import CacheNeed, CacheView, CompositeNeed, CompositeView, PagedKVNeed, PagedKVView, Runtime, SlotStateNeed, SlotStateView
+from ..parts.base import BorrowedKVNeed, CacheNeed, CacheView, CompositeNeed, CompositeView, PagedKVNeed, PagedKVView, Runtime, SlotStateNeed, SlotStateView
 from .pages import OutOfPages, PagePool, SlotPool
 
 __all__ = ["CacheLayout", "CacheManager", "RequestCache", "flatten_needs", "plan_cache_layout"]
@@ -67,10 +69,34 @@ class CacheLayout:
 def flatten_needs(needs: list[CacheNeed | None], cache_from: list[int | None]) -> tuple[list[CacheNeed | None], list[int | None], list[object]]:
     """Composite needs taken apart: ``(cells, cache_from per cell, shape per entry)``.  An entry's shape
     is the index of its cell, or a (nested) list of such for a :class:`CompositeNeed`; an entry that reads
-    another entry's cache reads that entry's cells one by one."""
+    another entry's cache reads that entry's cells one by one, unless its need names what it borrows (:class:`BorrowedKVNeed`): it
+    then has the other cells to itself.  A paged cell's window is widened to its borrowers'."""
     cells: list[CacheNeed | None] = []
     cell_from: list[int | None] = []
     shapes: list[object] = []
+
+    def paged_cells(shape: object) -> list[int]:
+        if isinstance(shape, list):
+            return [cell for part in shape for cell in paged_cells(part)]
+        return [shape] if isinstance(cells[shape], PagedKVNeed) else []
+
+    def borrows(need: CacheNeed | None) -> bool:
+        return any(borrows(part) for part in need.needs) if isinstance(need, CompositeNeed) else isinstance(need, BorrowedKVNeed)
+
+    def lay_borrowing(need: CacheNeed | None, source: object) -> object:
+        if isinstance(need, CompositeNeed):
+            return [lay_borrowing(part, source) for part in need.needs]
+        if not isinstance(need, BorrowedKVNeed):
+            return lay(need, None)
+        owners = paged_cells(source)
+        if len(owners) != 1 or cell_from[owners[0]] is not None:
+            raise ValueError("a schedule entry borrows the keys and values of an entry that does not hold exactly one set of its own")
+        owner = cells[owners[0]]
+        window = None if owner.window is None or need.window is None else max(owner.window, need.window)
+        cells[owners[0]] = replace(owner, window=window, keep_first=max(owner.keep_first, need.keep_first))
+        cells.append(need)
+        cell_from.append(owners[0])
+        return len(cells) - 1
 
     def lay(need: CacheNeed | None, source: object) -> object:
         if isinstance(need, CompositeNeed):
@@ -85,7 +111,12 @@ def flatten_needs(needs: list[CacheNeed | None], cache_from: list[int | None]) -
 
     for index, need in enumerate(needs):
         source = cache_from[index]
-        shapes.append(lay(need, None if source is None else shapes[source]))
+        if borrows(need):
+            if source is None:
+                raise ValueError(f"schedule entry {index} borrows keys and values, but no entry is named to borrow them from")
+            shapes.append(lay_borrowing(need, shapes[source]))
+        else:
+            shapes.append(lay(need, None if source is None else shapes[source]))
     return cells, cell_from, shapes
 
 

@@ -2,16 +2,21 @@
 
 from .errors import ConfigError, UnknownArchitectureError
 from .lfm2 import Lfm2Config
+from .mozetar import MozetarConfig
 from .plan import (
     AttentionSpec,
     BlockSpec,
     DenseMLPSpec,
+    DifferentialSpec,
     FeedForwardSpec,
     GatedDeltaSpec,
     GatedMLPSpec,
+    HyperBlockSpec,
+    InputConvSpec,
     LatentAttentionSpec,
     LayerNormSpec,
     LinearAttentionSpec,
+    LlamaScaling,
     MixerSpec,
     ModelPlan,
     NormSpec,
@@ -19,12 +24,14 @@ from .plan import (
     ParallelMixerSpec,
     PooledWindowAttentionSpec,
     PositionSpec,
+    QueryTemperature,
     RMSNormSpec,
     RopeSpec,
     RoutedMLPSpec,
     SandwichBlockSpec,
     ScheduleEntry,
     ShortConvSpec,
+    StreamConnectionSpec,
     StreamMixSpec,
     YarnScaling,
 )
@@ -39,32 +46,40 @@ register_architecture("Vuvulorn", VuvulornConfig)
 register_architecture("Tudulix", TudulixConfig)
 register_architecture("Vivulorn", VivulornConfig)
 register_architecture("Zozenex", ZozenexConfig)
+register_architecture("Mozetar", MozetarConfig)
 
 __all__ = [
     "AttentionSpec",
     "BlockSpec",
     "ConfigError",
     "DenseMLPSpec",
+    "DifferentialSpec",
     "FeedForwardSpec",
     "GatedDeltaSpec",
     "GatedMLPSpec",
+    "HyperBlockSpec",
+    "InputConvSpec",
     "LatentAttentionSpec",
     "LayerNormSpec",
     "Lfm2Config",
     "LinearAttentionSpec",
+    "LlamaScaling",
     "MixerSpec",
     "ModelPlan",
+    "MozetarConfig",
     "NormSpec",
     "OutputNormBlockSpec",
     "ParallelMixerSpec",
     "PooledWindowAttentionSpec",
     "PositionSpec",
+    "QueryTemperature",
     "RMSNormSpec",
     "RopeSpec",
     "RoutedMLPSpec",
     "SandwichBlockSpec",
     "ScheduleEntry",
     "ShortConvSpec",
+    "StreamConnectionSpec",
     "StreamMixSpec",
     "TudulixConfig",
     "UnknownArchitectureError",

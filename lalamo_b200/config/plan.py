@@ -20,14 +20,18 @@ __all__ = [
     "AttentionSpec",
     "BlockSpec",
     "DenseMLPSpec",
+    "DifferentialSpec",
     "EmbeddingSpec",
     "HeadSpec",
     "FeedForwardSpec",
     "GatedDeltaSpec",
     "GatedMLPSpec",
+    "HyperBlockSpec",
+    "InputConvSpec",
     "LatentAttentionSpec",
     "LayerNormSpec",
     "LinearAttentionSpec",
+    "LlamaScaling",
     "MixerSpec",
     "ModelPlan",
     "NormSpec",
@@ -35,12 +39,14 @@ __all__ = [
     "ParallelMixerSpec",
     "PooledWindowAttentionSpec",
     "PositionSpec",
+    "QueryTemperature",
     "RMSNormSpec",
     "RopeSpec",
     "RoutedMLPSpec",
     "SandwichBlockSpec",
     "ScheduleEntry",
     "ShortConvSpec",
+    "StreamConnectionSpec",
     "StreamMixSpec",
     "YarnScaling",
 ]
@@ -100,8 +106,20 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class LlamaScaling:
+    """Frequencies slowed down for contexts beyond the ``original`` one by wavelength ``l = 2 pi / f``: kept where ``l < original / high``,
+    divided by ``factor`` where ``l > original / low``, and between the two ``(1 - s) f / factor + s f`` with
+    ``s = (original / l - low) / (high - low)`` (the rule of Llama 3.1)."""
+
+    factor: float = 1.0
+    low: float = 1.0
+    high: float = 4.0
+    original: float = 8192.0
+
+
+@dataclass(frozen=True)
 class RopeSpec(PositionSpec):
-    """Unscaled rotary embedding over the first ``rotary_dim`` channels of a head
+    """Rotary embedding over the first ``rotary_dim`` channels of a head
     (``lalamo/modules/rope.py:58-102``).  ``pairing``: ``"half"`` rotates channel ``i`` with channel
     ``i + rotary_dim / 2`` (NeoX), ``"interleaved"`` channel ``2i`` with ``2i + 1``; pair ``i`` turns by
     ``position * theta ** (-2i / rotary_dim)`` either way."""
@@ -110,12 +128,33 @@ class RopeSpec(PositionSpec):
     rotary_dim: int = 0
     theta: float = 10000.0
     pairing: str = "half"
-    scaling: YarnScaling | None = None  # stretched frequencies and a factor on sines and cosines
+    # stretched frequencies (and, under YarnScaling, a factor on sines and cosines)
+    scaling: YarnScaling | LlamaScaling | None = None
 
 
 @dataclass(frozen=True)
 class MixerSpec:
     kind: ClassVar[str] = "abstract"
+
+
+@dataclass(frozen=True)
+class QueryTemperature:
+    """Queries grow with their position: times ``1 + coefficient * ln(floor((position + 1) / every) + 1)``."""
+
+    coefficient: float = 0.0
+    every: int = 1
+
+
+@dataclass(frozen=True)
+class DifferentialSpec:
+    """Attention as the difference of two maps over the same values.  A query head and a key head have two halves of ``head_dim``
+    channels, ``[map 1, map 2]``; with ``a1`` and ``a2`` the maps' outputs of a head, ``o = a1 - lambda a2``, ``lambda = exp(lq1 . lk1) -
+    exp(lq2 . lk2) + offset`` (four learned vectors of ``head_dim`` elements, one lambda for the layer), then ``o / sqrt(mean(o^2) + norm_eps)
+    * (1 - offset)`` over the head's channels.  ``head_gate``: times ``sigmoid(W_g h)``, one number per head."""
+
+    offset: float = 0.0
+    norm_eps: float = 1e-5
+    head_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -140,6 +179,13 @@ class AttentionSpec(MixerSpec):
     # between the norm and the rotation.
     qk_norm_whole: bool = False
     gated: bool = False  # the concatenated heads are multiplied by ``sigmoid(W_gate h)`` before the out-projection
+    differential: DifferentialSpec | None = None
+    query_temperature: QueryTemperature | None = None
+    # > 0: the projected q, k and v pass a causal depthwise convolution of so many taps before anything else (no bias, no activation)
+    conv_taps: int = 0
+    # True: the mixer has no keys and values of its own; it reads those that the schedule entry named by ``cache_from`` writes (with
+    # its own queries, window and scale)
+    borrows_kv: bool = False
 
 
 @dataclass(frozen=True)
@@ -205,7 +251,10 @@ class LinearAttentionSpec(MixerSpec):
     token, one number per head and key channel (``decay="channel"``): ``a = sigmoid(z) ** (1 / tau)`` with
     ``z = W_a2 (W_a1 h) + b`` through a bottleneck of ``decay_rank``.  Each head's read-out is divided by its root mean
     square (``norm_eps``; times a weight of ``value_dim`` elements shared by the heads if ``norm_weight``), the heads are
-    multiplied by ``silu(W_g h)`` (or ``sigmoid``, ``gate_activation``) and projected out.  State, decays and their logarithms,
+    multiplied by ``silu(W_g h)`` (or ``sigmoid``, ``gate_activation``; ``"none"``: no gate) and projected out.  ``decay="forget"``
+    (HGRN2): one forget gate per head and key channel, ``a = l + (1 - l) sigmoid(W_f h + b)`` with a learned lower bound ``l``, which
+    also says what is written, ``k = 1 - a`` (there is no key projection).  ``scaled="none"``: neither is scaled;
+    ``query_activation="silu"``: q is silu of its projection.  State, decays and their logarithms,
     the recurrence's inputs and the read-out norm are 32-bit."""
 
     kind: ClassVar[str] = "linear_attention"
@@ -221,6 +270,7 @@ class LinearAttentionSpec(MixerSpec):
     norm_weight: bool = False
     norm_eps: float = 1e-5
     gate_activation: str = "silu"
+    query_activation: str = "identity"
 
 
 @dataclass(frozen=True)
@@ -291,20 +341,22 @@ class GatedMLPSpec(FeedForwardSpec):
 @dataclass(frozen=True)
 class DenseMLPSpec(FeedForwardSpec):
     """``down(act(up(x) + b_up)) + b_down``: two projections, no gate.  ``activation``: ``"gelu"`` (the exact gelu,
-    ``0.5 z (1 + erf(z / sqrt 2))``), ``"silu"`` or ``"identity"``."""
+    ``0.5 z (1 + erf(z / sqrt 2))``), ``"silu"``, ``"identity"``, or ``"poly_norm"``: ``a N(z) + b N(z^2) + c N(z^3) + e`` with four learned
+    numbers, powers element by element and ``N(v) = v / sqrt(mean(v^2) + norm_eps)`` over a token's hidden values."""
 
     kind: ClassVar[str] = "dense_mlp"
     model_dim: int = 0
     hidden_dim: int = 0
     activation: str = "gelu"
     has_bias: bool = True
+    norm_eps: float = 1e-5  # of the "poly_norm" activation
 
 
 @dataclass(frozen=True)
 class RoutedMLPSpec(FeedForwardSpec):
     """A mixture of ``num_experts`` gated feed-forward layers of width ``hidden_dim`` of which each token
     uses ``top``: router scores ``score(W_router h)`` in 32-bit; experts in ``group_count`` equal groups of
-    neighbours, a group scored by the sum of its two largest scores, only the best ``group_keep`` groups
+    neighbours, a group scored by the sum of its two largest scores (``group_score="largest"``: by its largest), only the best ``group_keep`` groups
     eligible; the chosen scores (over their sum if ``renormalize``) weigh the experts' outputs.
     ``router_bias``: a bias on the router's logits.  ``score="logits"`` ranks experts by the logits themselves;
     ``chosen_softmax``: the weights are the softmax over the chosen scores only.  ``limit``: of the experts'
@@ -331,6 +383,40 @@ class RoutedMLPSpec(FeedForwardSpec):
     choice_bias: bool = False
     weight_scale: float = 1.0
     shared_gate: bool = False
+    group_score: str = "two_largest"
+
+
+@dataclass(frozen=True)
+class InputConvSpec:
+    """What a sublayer reads, ``h``, becomes ``h + conv(h)``: a causal depthwise convolution of ``taps`` taps, no bias."""
+
+    kind: ClassVar[str] = "input_conv"
+    model_dim: int = 0
+    taps: int = 1
+
+
+@dataclass(frozen=True)
+class StreamConnectionSpec:
+    """How a sublayer reads from and writes to ``streams`` parallel residual streams (hyper-connections): it reads
+    ``u = sum_s read[s] X_s``, and its output ``y`` turns all streams at once into ``X_to <- sum_from mix[from, to] X_from + write[to] y``."""
+
+    kind: ClassVar[str] = "stream_connection"
+    streams: int = 1
+
+
+@dataclass(frozen=True)
+class HyperBlockSpec:
+    """A pre-norm block on parallel residual streams: each sublayer reads the norm of what its connection reads and writes through
+    its connection; the mixer's input may pass a causal convolution first (``ffn=None``: no second half)."""
+
+    pre_mixer_norm: NormSpec
+    mixer: MixerSpec
+    mixer_connection: StreamConnectionSpec
+    input_conv: InputConvSpec | None = None
+    pre_ffn_norm: NormSpec | None = None
+    ffn: FeedForwardSpec | None = None
+    ffn_connection: StreamConnectionSpec | None = None
+    arrangement: str = "hyper"
 
 
 @dataclass(frozen=True)
@@ -412,7 +498,8 @@ class ScheduleEntry:
     ``layer`` indexes ``ModelPlan.layers`` (a layer may appear in several entries).
     ``cache_from`` names an earlier schedule entry whose cache this execution reads
     instead of owning one (the reference's ``kv_source_layer_index``,
-    ``lalamo/modules/transformer.py:210-217``).
+    ``lalamo/modules/transformer.py:210-217``).  A mixer that borrows only part of it (keys and values, beside state of
+    its own) says so in its own need.
     """
 
     layer: int
@@ -429,7 +516,7 @@ class ScheduleEntry:
 class ModelPlan:
     vocab_size: int
     model_dim: int
-    layers: tuple[BlockSpec | OutputNormBlockSpec | SandwichBlockSpec, ...]
+    layers: tuple[BlockSpec | HyperBlockSpec | OutputNormBlockSpec | SandwichBlockSpec, ...]
     final_norm: NormSpec
     tie_embeddings: bool = True
     embedding_scale: float | None = None
@@ -440,6 +527,9 @@ class ModelPlan:
     embedding: EmbeddingSpec | None = None
     head: HeadSpec | None = None
     stream_mix: StreamMixSpec | None = None  # needed by schedule entries with ``mix_embedding``
+    # > 0: the residual is this many parallel streams, all equal to the embedding's output at first, whose sum the final norm reads;
+    # every layer is then a :class:`HyperBlockSpec`
+    streams: int = 0
 
     def __post_init__(self) -> None:
         if self.embedding is None:
@@ -450,7 +540,12 @@ class ModelPlan:
             object.__setattr__(
                 self, "schedule", tuple(ScheduleEntry(i) for i in range(len(self.layers)))
             )
+        hyper = [isinstance(layer, HyperBlockSpec) for layer in self.layers]
+        if any(hyper) != (self.streams > 0) or (self.streams > 0 and not all(hyper)):
+            raise ValueError("parallel residual streams and blocks that read and write such streams go together")
         for position, entry in enumerate(self.schedule):
+            if self.streams > 0 and (entry.add_embedding or entry.mix_embedding):
+                raise ValueError(f"schedule[{position}] feeds the embedding again, which parallel streams do not support")
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"schedule[{position}] names layer {entry.layer}, but there are {len(self.layers)}")
             if entry.mix_embedding and self.stream_mix is None:

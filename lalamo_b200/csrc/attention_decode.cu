@@ -12,6 +12,11 @@
 //   * keys: column n of 8-key block b stands for key 4*(n/2) + 2*b + n%2 of the 16, so that lane t
 //     holds probabilities of keys 4t..4t+3, which are contiguous in the transposed value page.
 // Keys are [page][row][group][hd]; values are transposed, [page][group][hd][row]; page_size % 16 == 0.
+// Kernels with GENERAL = false take key and value heads of HD channels each; with GENERAL = true key heads of up to HD channels (a
+// multiple of 16), value heads of up to HD (a multiple of 8), several key heads over one value head, float32 output, and rows of the
+// cache that hold the keys of two attention maps side by side: a group's query heads are then those of the first map, which
+// meet the row's first half, and those of the second, which meet its second half (their other half counts as zeros), so that
+// both maps read keys and values once.
 // Partial results (max, sum, unnormalised output per split) go to scratch; a second kernel merges
 // them in split order, so the result does not depend on the batch or on the grid.
 #include "common.cuh"
@@ -45,8 +50,8 @@ struct DecodeParams {
     const __nv_bfloat16* q;         // [tokens, heads, hd]
     const __nv_bfloat16* k_pages;   // [pages, page_size, groups, hd]
     const __nv_bfloat16* v_pages;   // [pages, groups, hd, page_size]
-    __nv_bfloat16* out;             // [tokens, heads, hd]: written by this kernel itself when there is one split
-    float* partial_out;             // [tokens, heads, splits, hd]
+    void* out;                      // [tokens, heads, value_dim], bfloat16 or float32 (out_float): written by this kernel itself when there is one split
+    float* partial_out;             // [tokens, heads, splits, value_dim]
     float* partial_stats;           // [tokens, heads, splits, 2]  (max in base-2 units, sum)
     const int* positions;
     const int* token_segment;
@@ -61,6 +66,10 @@ struct DecodeParams {
     // >= 0: the kernel is launched to start before the kernel before it has finished, and the newest `fresh_keys`
     // positions a token sees may still be written by that kernel; it reads the older ones while it waits.
     int fresh_keys;
+    // GENERAL only (else key_dim = value_dim = HD, keys_per_value 1, the rest 0)
+    int key_dim, value_dim;   // channels of a cache row's keys (both maps' together with two_maps) and of a value head
+    int keys_per_value;       // key heads that share a value head
+    int two_maps, out_float;
 };
 
 // The page that holds 16-key block `key_block` of the request, or -1, and the block's first row in it.
@@ -83,20 +92,22 @@ struct DecodeLaneSources {
     int value_step;                 // elements from a lane's value row to its next (8 channels on)
 };
 
-template <int HD>
+template <int HD, bool GENERAL>
 __device__ __forceinline__ DecodeLaneSources decode_lane_sources(const DecodeParams& p, int group, int lane) {
     const int g = lane >> 2, t = lane & 3;
+    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
+    const int value_groups = GENERAL ? p.num_groups / p.keys_per_value : p.num_groups, value_group = GENERAL ? group / p.keys_per_value : group;
     DecodeLaneSources sources;
-    sources.key_row_stride = p.num_groups * HD;
+    sources.key_row_stride = p.num_groups * kd;
     sources.key_page_stride = static_cast<size_t>(p.page_size) * sources.key_row_stride;
-    sources.value_page_stride = static_cast<size_t>(p.num_groups) * HD * p.page_size;
+    sources.value_page_stride = static_cast<size_t>(value_groups) * vd * p.page_size;
     sources.value_step = 8 * p.page_size;
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
         const int key = 4 * (g >> 1) + 2 * b + (g & 1);
-        sources.keys[b] = p.k_pages + static_cast<size_t>(key) * sources.key_row_stride + group * HD + t * (HD / 4);
+        sources.keys[b] = p.k_pages + static_cast<size_t>(key) * sources.key_row_stride + group * kd + t * (kd / 4);
     }
-    sources.values = p.v_pages + (static_cast<size_t>(group) * HD + g) * p.page_size + 4 * t;
+    sources.values = p.v_pages + (static_cast<size_t>(value_group) * vd + g) * p.page_size + 4 * t;
     return sources;
 }
 
@@ -124,8 +135,8 @@ __device__ __forceinline__ void async_copy_8(void* shared_destination, const voi
 }
 
 // Starts the copies of a 16-key block (rows `in_page`.. of `page`; page -1: zeros) into `stage`.
-template <int HD>
-__device__ __forceinline__ void issue_fragments(unsigned char* stage, const DecodeLaneSources& sources, int page, int in_page, int lane, bool& bad) {
+template <int HD, bool GENERAL>
+__device__ __forceinline__ void issue_fragments(unsigned char* stage, const DecodeLaneSources& sources, int page, int in_page, int lane, int kd, int vd, bool& bad) {
     unsigned char* keys = stage;
     unsigned char* values = stage + HD * 32;
     if (page < 0) {
@@ -139,7 +150,12 @@ __device__ __forceinline__ void issue_fragments(unsigned char* stage, const Deco
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
         const __nv_bfloat16* row = sources.keys[b] + key_offset;
-        if constexpr (HD % 32 == 0) {
+        if constexpr (GENERAL) {
+#pragma unroll
+            for (int j = 0; j < HD / 16; ++j) {
+                if (16 * j < kd) async_copy_8(keys + ((b * (HD / 16) + j) * 32 + lane) * 8, reinterpret_cast<const uint2*>(row) + j);
+            }
+        } else if constexpr (HD % 32 == 0) {
 #pragma unroll
             for (int j = 0; j < HD / 32; ++j) async_copy_16(keys + ((b * (HD / 32) + j) * 32 + lane) * 16, reinterpret_cast<const uint4*>(row) + j);
         } else {
@@ -150,17 +166,18 @@ __device__ __forceinline__ void issue_fragments(unsigned char* stage, const Deco
     const __nv_bfloat16* source = sources.values + page * sources.value_page_stride + in_page;
 #pragma unroll
     for (int n = 0; n < HD / 8; ++n) {
+        if (GENERAL && 8 * n >= vd) break;
         async_copy_8(values + (n * 32 + lane) * 8, source);
         source += sources.value_step;
     }
 }
 
 // Reads this lane's key fragments of a stage whose copies have arrived: k[8-key block][channel block][b0, b1].
-template <int HD>
+template <int HD, bool GENERAL>
 __device__ __forceinline__ void read_key_fragments(uint32_t (&k)[2][HD / 16][2], const unsigned char* stage, int lane) {
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
-        if constexpr (HD % 32 == 0) {
+        if constexpr (HD % 32 == 0 && !GENERAL) {
 #pragma unroll
             for (int j = 0; j < HD / 32; ++j) {
                 const uint4 loaded = *reinterpret_cast<const uint4*>(stage + ((b * (HD / 32) + j) * 32 + lane) * 16);
@@ -193,7 +210,7 @@ __device__ __forceinline__ void read_value_fragments(uint32_t (&v)[HD / 8][2], c
 }
 
 // grid (splits, groups * row_tiles, tokens), kDecodeWarps warps.
-template <int HD>
+template <int HD, bool GENERAL>
 __global__ void __launch_bounds__(kDecodeWarps * 32, HD <= 64 ? 4 : 1)   // head size 64: 128 registers, four CTAs per SM
 attention_decode_kernel(const DecodeParams p) {
     const int split = blockIdx.x, place = blockIdx.z;
@@ -219,6 +236,7 @@ attention_decode_kernel(const DecodeParams p) {
     const int end = min(begin + p.blocks_per_split, kept_blocks + last_block - first_block + 1);
     const int rows_here = min(16, heads_per_group - row_tile * 16);
     const int head_base = group * heads_per_group + row_tile * 16;
+    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
 
     uint32_t q_frag[HD / 16][4];
     float out[HD / 8][4];
@@ -233,7 +251,7 @@ attention_decode_kernel(const DecodeParams p) {
     extern __shared__ __align__(16) unsigned char ring_memory[];
     unsigned char* ring = ring_memory + warp * Ring::kWarpBytes;
     const int count = end > begin + warp ? (end - begin - warp + kDecodeWarps - 1) / kDecodeWarps : 0;   // this warp's blocks: begin + warp + 4 i
-    const DecodeLaneSources sources = decode_lane_sources<HD>(p, group, lane);
+    const DecodeLaneSources sources = decode_lane_sources<HD, GENERAL>(p, group, lane);
     int table_first = 0;
     int lane_in_page = 0;
     int lane_page = lane < count ? decode_page_of(p, segment, block_of(begin + warp + kDecodeWarps * lane), lane_in_page) : -1;
@@ -245,8 +263,8 @@ attention_decode_kernel(const DecodeParams p) {
                 table_first = issued;
                 lane_page = issued + lane < count ? decode_page_of(p, segment, block_of(begin + warp + kDecodeWarps * (issued + lane)), lane_in_page) : -1;
             }
-            issue_fragments<HD>(ring + issue_stage * Ring::kStageBytes, sources, __shfl_sync(0xffffffffu, lane_page, issued - table_first),
-                                __shfl_sync(0xffffffffu, lane_in_page, issued - table_first), lane, bad);
+            issue_fragments<HD, GENERAL>(ring + issue_stage * Ring::kStageBytes, sources, __shfl_sync(0xffffffffu, lane_page, issued - table_first),
+                                __shfl_sync(0xffffffffu, lane_in_page, issued - table_first), lane, kd, vd, bad);
             ++issued;
             issue_stage = issue_stage + 1 == Ring::kStages ? 0 : issue_stage + 1;
         }
@@ -270,7 +288,14 @@ attention_decode_kernel(const DecodeParams p) {
         for (int half = 0; half < 2; ++half) {
             const int row = g + 8 * half;
             uint2 loaded = make_uint2(0u, 0u);
-            if (row < rows_here) {
+            if constexpr (GENERAL) {
+                // with two maps a query head has half as many channels as the cache row, and meets its map's half of it
+                const int map = p.two_maps ? 2 * (row_tile * 16 + row) / heads_per_group : 0, q_dim = p.two_maps ? kd / 2 : kd;
+                if (row < rows_here && 16 * j < kd && (!p.two_maps || map == t >> 1)) {
+                    const __nv_bfloat16* src = p.q + (static_cast<size_t>(token) * p.num_heads + head_base + row) * q_dim + t * (kd / 4) - map * q_dim + 4 * j;
+                    loaded = *reinterpret_cast<const uint2*>(src);
+                }
+            } else if (row < rows_here) {
                 const __nv_bfloat16* src = p.q + (static_cast<size_t>(token) * p.num_heads + head_base + row) * HD + t * (HD / 4) + 4 * j;
                 loaded = *reinterpret_cast<const uint2*>(src);
             }
@@ -298,11 +323,13 @@ attention_decode_kernel(const DecodeParams p) {
             for (int b = 0; b < 2; ++b) s[which][b][0] = s[which][b][1] = s[which][b][2] = s[which][b][3] = which == 1 && !two ? -INFINITY : 0.0f;
             if (which == 0 || two) {
                 uint32_t k[2][HD / 16][2];
-                read_key_fragments<HD>(k, stages[which], lane);
+                read_key_fragments<HD, GENERAL>(k, stages[which], lane);
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
 #pragma unroll
-                    for (int j = 0; j < HD / 16; ++j) mma_16816(s[which][b], q_frag[j], k[b][j][0], k[b][j][1]);
+                    for (int j = 0; j < HD / 16; ++j) {
+                        if (!GENERAL || 16 * j < kd) mma_16816(s[which][b], q_frag[j], k[b][j][0], k[b][j][1]);
+                    }
                 }
             }
         }
@@ -393,7 +420,9 @@ attention_decode_kernel(const DecodeParams p) {
                     }
                 }
 #pragma unroll
-                for (int n = 0; n < HD / 8; ++n) mma_16816(out[n], p_frag[which], v[n][0], v[n][1]);
+                for (int n = 0; n < HD / 8; ++n) {
+                    if (!GENERAL || 8 * n < vd) mma_16816(out[n], p_frag[which], v[n][0], v[n][1]);
+                }
             }
         }
         issue_next();
@@ -425,8 +454,8 @@ attention_decode_kernel(const DecodeParams p) {
         shared_sum[warp][g + 8] = row_sum[1];
     }
     __syncthreads();
-    for (int index = threadIdx.x; index < rows_here * HD; index += blockDim.x) {
-        const int row = index / HD, d = index - row * HD;
+    for (int index = threadIdx.x; index < rows_here * vd; index += blockDim.x) {
+        const int row = index / vd, d = index - row * vd;
         float merged_max = -INFINITY;
 #pragma unroll
         for (int w = 0; w < kDecodeWarps; ++w) merged_max = fmaxf(merged_max, shared_max[w][row]);
@@ -439,11 +468,14 @@ attention_decode_kernel(const DecodeParams p) {
         }
         if (p.splits == 1) {
             // all of the token's keys were this CTA's: what the merge kernel would make of the one partial
-            p.out[(static_cast<size_t>(token) * p.num_heads + head_base + row) * HD + d] = __float2bfloat16_rn(sum > 0.0f ? value / sum : 0.0f);
+            const size_t place_out = (static_cast<size_t>(token) * p.num_heads + head_base + row) * vd + d;
+            const float result = sum > 0.0f ? value / sum : 0.0f;
+            if (GENERAL && p.out_float) static_cast<float*>(p.out)[place_out] = result;
+            else static_cast<__nv_bfloat16*>(p.out)[place_out] = __float2bfloat16_rn(result);
             continue;
         }
         const size_t slot = (static_cast<size_t>(place) * p.num_heads + head_base + row) * p.splits + split;
-        p.partial_out[slot * HD + d] = value;
+        p.partial_out[slot * vd + d] = value;
         if (d == 0) {
             p.partial_stats[slot * 2] = merged_max;
             p.partial_stats[slot * 2 + 1] = sum;
@@ -453,9 +485,10 @@ attention_decode_kernel(const DecodeParams p) {
 
 // grid (heads, tokens); merges the splits in order and normalises.  The partials of up to eight
 // splits are asked for together (one after the other, every split would cost a trip to L2).
-template <int HD>
+template <int HD, typename TO>   // HD 0: any size of a value head, given in `value_dim`
 __global__ void attention_decode_merge_kernel(const float* __restrict__ partial_out, const float* __restrict__ partial_stats,
-                                              __nv_bfloat16* __restrict__ out, const int* __restrict__ token_list, int num_heads, int splits) {
+                                              TO* __restrict__ out, const int* __restrict__ token_list, int num_heads, int splits, int value_dim) {
+    const int vd = HD > 0 ? HD : value_dim;
     allow_next_kernel();   // the out-projection that follows may start pulling its weights towards L2
     const int head = blockIdx.x, place = blockIdx.y;
     const int token = token_list ? token_list[place] : place;
@@ -469,7 +502,7 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ partial_
 #pragma unroll
         for (int i = 0; i < kBatch; ++i) merged_max = fmaxf(merged_max, maxima[i]);
     }
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    for (int d = threadIdx.x; d < vd; d += blockDim.x) {
         float value = 0.0f, sum = 0.0f;
         for (int first = 0; first < splits; first += kBatch) {
             float maxima[kBatch], sums[kBatch], values[kBatch];
@@ -478,7 +511,7 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ partial_
                 const bool here = first + i < splits;
                 maxima[i] = here ? partial_stats[(base + first + i) * 2] : -INFINITY;
                 sums[i] = here ? partial_stats[(base + first + i) * 2 + 1] : 0.0f;
-                values[i] = here ? partial_out[(base + first + i) * HD + d] : 0.0f;
+                values[i] = here ? partial_out[(base + first + i) * vd + d] : 0.0f;
             }
 #pragma unroll
             for (int i = 0; i < kBatch; ++i) {   // in split order
@@ -487,16 +520,16 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ partial_
                 sum += sums[i] * weight;
             }
         }
-        out[(static_cast<size_t>(token) * num_heads + head) * HD + d] = __float2bfloat16_rn(sum > 0.0f ? value / sum : 0.0f);
+        out[(static_cast<size_t>(token) * num_heads + head) * vd + d] = from_float<TO>(sum > 0.0f ? value / sum : 0.0f);
     }
 }
 
-template <int HD>
-int launch_decode(const DecodeParams& p, __nv_bfloat16* out, int tokens, cudaStream_t stream) {
+template <int HD, bool GENERAL>
+int launch_decode(const DecodeParams& p, int tokens, cudaStream_t stream) {
     const int heads_per_group = p.num_heads / p.num_groups;
     const int row_tiles = (heads_per_group + 15) / 16;
     const dim3 grid(p.splits, p.num_groups * row_tiles, tokens);
-    auto kernel = attention_decode_kernel<HD>;
+    auto kernel = attention_decode_kernel<HD, GENERAL>;
     static OncePerDevice configured;
     if (allow_shared_memory(configured, kernel, DecodeRing<HD>::kBytes) != cudaSuccess) return static_cast<int>(cudaGetLastError());
     if (p.fresh_keys >= 0) {
@@ -505,9 +538,18 @@ int launch_decode(const DecodeParams& p, __nv_bfloat16* out, int tokens, cudaStr
     } else {
         kernel<<<grid, kDecodeWarps * 32, DecodeRing<HD>::kBytes, stream>>>(p);
     }
-    if (p.splits > 1)
-        attention_decode_merge_kernel<HD><<<dim3(p.num_heads, tokens), HD >= 64 ? 64 : 32, 0, stream>>>(p.partial_out, p.partial_stats, out,
-                                                                                                      p.token_list, p.num_heads, p.splits);
+    if (p.splits > 1) {
+        const dim3 merge_grid(p.num_heads, tokens);
+        if (GENERAL && p.out_float)
+            attention_decode_merge_kernel<0, float><<<merge_grid, 64, 0, stream>>>(p.partial_out, p.partial_stats, static_cast<float*>(p.out), p.token_list, p.num_heads,
+                                                                                 p.splits, p.value_dim);
+        else if (GENERAL)
+            attention_decode_merge_kernel<0, __nv_bfloat16><<<merge_grid, 64, 0, stream>>>(p.partial_out, p.partial_stats, static_cast<__nv_bfloat16*>(p.out),
+                                                                                         p.token_list, p.num_heads, p.splits, p.value_dim);
+        else
+            attention_decode_merge_kernel<HD, __nv_bfloat16><<<merge_grid, HD >= 64 ? 64 : 32, 0, stream>>>(
+                p.partial_out, p.partial_stats, static_cast<__nv_bfloat16*>(p.out), p.token_list, p.num_heads, p.splits, HD);
+    }
     return static_cast<int>(cudaGetLastError());
 }
 
@@ -523,8 +565,8 @@ int lb_attention_decode_ctas_per_sm(int head_dim) {
 #define LB_DECODE_OCCUPANCY(HD)                                                                                          \
     case HD: {                                                                                                           \
         static lb::OncePerDevice configured;                                                                             \
-        if (lb::allow_shared_memory(configured, lb::attention_decode_kernel<HD>, lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0; \
-        if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&ctas, lb::attention_decode_kernel<HD>, lb::kDecodeWarps * 32,  \
+        if (lb::allow_shared_memory(configured, lb::attention_decode_kernel<HD, false>, lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0; \
+        if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&ctas, lb::attention_decode_kernel<HD, false>, lb::kDecodeWarps * 32,  \
                                                           lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0;          \
         return ctas;                                                                                                     \
     }
@@ -536,30 +578,43 @@ int lb_attention_decode_ctas_per_sm(int head_dim) {
 #undef LB_DECODE_OCCUPANCY
 }
 
-// Floats of scratch the call needs: tokens * heads * splits * (head_dim + 2).  `tokens` counts the
+// Floats of scratch the call needs: tokens * heads * splits * (value size + 2).  `tokens` counts the
 // tokens that run: the length of `token_list`, or all tokens when it is null.
 long long lb_attention_decode_scratch_floats(int tokens, int num_heads, int head_dim, int splits) {
     return static_cast<long long>(tokens) * num_heads * splits * (head_dim + 2);
 }
 
 // Returns 0, a CUDA error code, -1 for an unsupported type, or -2 for sizes the kernel does not take
-// (head_dim must be a multiple of 16 up to 128, page_size a multiple of 16, the scale positive).
+// (head_dim must be a multiple of 16 up to 128, page_size a multiple of 16, the scale positive).  value_dim (0: head_dim), value_groups
+// (0: num_groups), two_maps and out_float: see GENERAL above; with two_maps head_dim counts both maps' channels, num_groups the
+// cache rows' groups and num_heads both maps' query heads; value_dim must be a multiple of 8 up to 128.
 int lb_attention_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* scratch,
                         const int* positions, const int* token_segment, const int* block_table, const int* token_list,
                         int tokens, int num_heads, int num_groups, int head_dim, int page_size, int num_pages, int max_blocks,
                         float scale, int window, int splits, int blocks_per_split, int fresh_keys, int* status, cudaStream_t stream,
-                        int keep_first) {
+                        int keep_first, int value_dim, int value_groups, int two_maps, int out_float) {
     // fresh_keys >= 0: see DecodeParams (the caller's previous kernel on the stream writes at most that many of
     // the newest positions a token sees, and lets this kernel start early); -1: an ordinary launch.
     if (tokens == 0) return 0;
     if (page_size % 16 != 0 || num_heads % num_groups != 0 || splits < 1 || blocks_per_split < 1 || !(scale > 0.0f) || fresh_keys < -1 || keep_first < 0) return -2;
+    if (value_dim <= 0) value_dim = head_dim;
+    if (value_groups <= 0) value_groups = num_groups;
+    const bool general = value_dim != head_dim || value_groups != num_groups || two_maps || out_float;
+    if (general && (head_dim % 16 != 0 || head_dim < 16 || head_dim > 128 || value_dim % 8 != 0 || value_dim < 8 || value_dim > 128 || num_groups % value_groups != 0 ||
+                    (two_maps && (num_heads / num_groups) % 2 != 0)))
+        return -2;
     lb::DecodeParams p;
     p.q = static_cast<const __nv_bfloat16*>(q);
     p.k_pages = static_cast<const __nv_bfloat16*>(k_pages);
     p.v_pages = static_cast<const __nv_bfloat16*>(v_pages);
-    p.out = static_cast<__nv_bfloat16*>(out);
+    p.out = out;
+    p.key_dim = head_dim;
+    p.value_dim = value_dim;
+    p.keys_per_value = num_groups / value_groups;
+    p.two_maps = two_maps;
+    p.out_float = out_float;
     p.partial_out = scratch;
-    p.partial_stats = scratch + static_cast<size_t>(tokens) * num_heads * splits * head_dim;
+    p.partial_stats = scratch + static_cast<size_t>(tokens) * num_heads * splits * value_dim;
     p.positions = positions;
     p.token_segment = token_segment;
     p.block_table = block_table;
@@ -576,16 +631,22 @@ int lb_attention_decode(const void* q, const void* k_pages, const void* v_pages,
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
     p.fresh_keys = fresh_keys;
-    __nv_bfloat16* result = static_cast<__nv_bfloat16*>(out);
+    if (general) {
+        const int widest = head_dim > value_dim ? head_dim : value_dim;
+        if (widest <= 32) return lb::launch_decode<32, true>(p, tokens, stream);
+        if (widest <= 64) return lb::launch_decode<64, true>(p, tokens, stream);
+        if (widest <= 96) return lb::launch_decode<96, true>(p, tokens, stream);
+        return lb::launch_decode<128, true>(p, tokens, stream);
+    }
     switch (head_dim) {
-        case 16: return lb::launch_decode<16>(p, result, tokens, stream);
-        case 32: return lb::launch_decode<32>(p, result, tokens, stream);
-        case 48: return lb::launch_decode<48>(p, result, tokens, stream);
-        case 64: return lb::launch_decode<64>(p, result, tokens, stream);
-        case 80: return lb::launch_decode<80>(p, result, tokens, stream);
-        case 96: return lb::launch_decode<96>(p, result, tokens, stream);
-        case 112: return lb::launch_decode<112>(p, result, tokens, stream);
-        case 128: return lb::launch_decode<128>(p, result, tokens, stream);
+        case 16: return lb::launch_decode<16, false>(p, tokens, stream);
+        case 32: return lb::launch_decode<32, false>(p, tokens, stream);
+        case 48: return lb::launch_decode<48, false>(p, tokens, stream);
+        case 64: return lb::launch_decode<64, false>(p, tokens, stream);
+        case 80: return lb::launch_decode<80, false>(p, tokens, stream);
+        case 96: return lb::launch_decode<96, false>(p, tokens, stream);
+        case 112: return lb::launch_decode<112, false>(p, tokens, stream);
+        case 128: return lb::launch_decode<128, false>(p, tokens, stream);
         default: return -2;
     }
 }
@@ -665,7 +726,7 @@ extern "C" int lb_attention_decode_static(const void* q, const void* k_pages, co
     // Every partial slot of this call is written by the first kernel before the second reads it, so
     // nothing left over from an earlier call needs clearing.
     const int code = lb_attention_decode(q, k_pages, v_pages, out, scratch, positions, token_segment, block_table, token_list, tokens, num_heads,
-                                         num_groups, head_dim, page_size, num_pages, max_blocks, scale, window, splits, blocks_per_split, -1, status, stream, 0);
+                                         num_groups, head_dim, page_size, num_pages, max_blocks, scale, window, splits, blocks_per_split, -1, status, stream, 0, 0, 0, 0, 0);
     if (code == -2) lb::describe(error_message, error_capacity, "attention_decode_static: head_dim must be a multiple of 16 up to 128 and page_size a multiple of 16");
     else if (code != 0) lb::describe(error_message, error_capacity, "attention_decode_static: launch failed with CUDA error %lld", code);
     return code;

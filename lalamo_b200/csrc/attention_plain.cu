@@ -15,6 +15,7 @@ struct PagedLayout {
     int num_groups;   // K/V heads
     int head_dim;     // channels of a query or key head
     int value_dim;    // channels of a value head
+    int value_groups; // value heads: as many as key heads, or a divisor of them (consecutive key heads then share a value head)
 };
 
 // Keys are stored [page][row][group][head_dim]; values transposed, [page][group][head_dim][row], so
@@ -34,7 +35,7 @@ __device__ __forceinline__ T* page_row(T* pages, const int* block_table, const P
     return pages + (row * layout.num_groups + group) * layout.head_dim;
 }
 
-// Address of channel 0 of the value of `position`; channel d lies `d * page_size` elements further.
+// Address of channel 0 of the value of `position` in value head `group`; channel d lies `d * page_size` elements further.
 template <typename T>
 __device__ __forceinline__ T* value_column(T* pages, const int* block_table, const PagedLayout& layout, int segment,
                                            int position, int group) {
@@ -42,7 +43,7 @@ __device__ __forceinline__ T* value_column(T* pages, const int* block_table, con
     if (block >= layout.max_blocks) return nullptr;
     const int page = block_table[static_cast<size_t>(segment) * layout.max_blocks + block];
     if (page < 0 || page >= layout.num_pages) return nullptr;
-    const size_t base = (static_cast<size_t>(page) * layout.num_groups + group) * layout.value_dim * layout.page_size;
+    const size_t base = (static_cast<size_t>(page) * layout.value_groups + group) * layout.value_dim * layout.page_size;
     return pages + base + (position - block * layout.page_size);
 }
 
@@ -55,7 +56,15 @@ struct RewriteExtras {
     float turn_scale;   // sines and cosines are multiplied by this
     int row_stride;     // elements between the rows of qkv (>= the q, k and v columns; what follows them is not read)
     int inline_whole;   // the warp-per-head kernel computes the projection-wide statistic itself (row_inv is then only a flag)
+    // Queries are multiplied by 1 + temperature * ln(floor((position + 1) / temperature_every) + 1) (temperature_every 0: they are not).
+    float temperature;
+    int temperature_every;
 };
+
+__device__ __forceinline__ float query_factor(const RewriteExtras& extra, int position) {
+    if (extra.temperature_every <= 0) return 1.0f;
+    return 1.0f + extra.temperature * logf(static_cast<float>((position + 1) / extra.temperature_every) + 1.0f);
+}
 
 // grid (tokens, num_heads + num_groups), one warp per head vector.
 //   y < num_heads: query head -> q_out[token, head, :]
@@ -95,16 +104,19 @@ __global__ void qk_norm_rope_write_kernel(const T* __restrict__ qkv, T* __restri
     } else {
         const int segment = token_segment[token];
         dst = page_row(k_pages, block_table, layout, segment, position, group);
-        T* v_dst = value_column(v_pages, block_table, layout, segment, position, group);
-        if (dst == nullptr || v_dst == nullptr) {
+        if (dst == nullptr) {
             if (lane == 0) report_error(status, kBadPage);
             return;
         }
-        const size_t v_offset = static_cast<size_t>(num_heads + layout.num_groups) * hd + static_cast<size_t>(group) * vd;
-        const T* v_src = qkv + static_cast<size_t>(token) * width + v_offset;
-        for (int d = lane; d < vd; d += 32)
-            v_dst[static_cast<size_t>(d) * layout.page_size] = bias ? from_float<T>(to_float(v_src[d]) + bias[v_offset + d]) : v_src[d];
+        if (group < layout.value_groups) {
+            T* v_dst = value_column(v_pages, block_table, layout, segment, position, group);
+            const size_t v_offset = static_cast<size_t>(num_heads + layout.num_groups) * hd + static_cast<size_t>(group) * vd;
+            const T* v_src = qkv + static_cast<size_t>(token) * width + v_offset;
+            for (int d = lane; d < vd; d += 32)
+                v_dst[static_cast<size_t>(d) * layout.page_size] = bias ? from_float<T>(to_float(v_src[d]) + bias[v_offset + d]) : v_src[d];
+        }
     }
+    const float factor = is_query ? query_factor(extra, position) : 1.0f;
 
     float inv = 1.0f;
     if (whole && extra.inline_whole) {
@@ -146,7 +158,7 @@ __global__ void qk_norm_rope_write_kernel(const T* __restrict__ qkv, T* __restri
             const float rotated = d < half ? -other : other;
             y = (y * cosine + rotated * sine) * extra.turn_scale;
         }
-        dst[d] = from_float<T>(y);
+        dst[d] = from_float<T>(y * factor);
     }
 }
 
@@ -194,16 +206,19 @@ __global__ void qk_norm_rope_write_token_kernel(const T* __restrict__ qkv, T* __
             dst = q_out + (static_cast<size_t>(token) * num_heads + unit) * hd;
         } else {
             dst = page_row(k_pages, block_table, layout, segment, position, group);
-            T* v_dst = value_column(v_pages, block_table, layout, segment, position, group);
-            if (dst == nullptr || v_dst == nullptr) {
+            if (dst == nullptr) {
                 if (lane == 0) report_error(status, kBadPage);
                 continue;
             }
-            const size_t v_offset = static_cast<size_t>(num_heads + layout.num_groups) * hd + static_cast<size_t>(group) * vd;
-            const T* v_src = qkv + static_cast<size_t>(token) * width + v_offset;
-            for (int d = lane; d < vd; d += 32)
-                v_dst[static_cast<size_t>(d) * layout.page_size] = bias ? from_float<T>(to_float(v_src[d]) + bias[v_offset + d]) : v_src[d];
+            if (group < layout.value_groups) {
+                T* v_dst = value_column(v_pages, block_table, layout, segment, position, group);
+                const size_t v_offset = static_cast<size_t>(num_heads + layout.num_groups) * hd + static_cast<size_t>(group) * vd;
+                const T* v_src = qkv + static_cast<size_t>(token) * width + v_offset;
+                for (int d = lane; d < vd; d += 32)
+                    v_dst[static_cast<size_t>(d) * layout.page_size] = bias ? from_float<T>(to_float(v_src[d]) + bias[v_offset + d]) : v_src[d];
+            }
         }
+        const float factor = is_query ? query_factor(extra, position) : 1.0f;
         float inv = 1.0f;
         if (whole) {
             inv = extra.row_inv[2 * static_cast<size_t>(token) + (is_query ? 0 : 1)];
@@ -229,7 +244,7 @@ __global__ void qk_norm_rope_write_token_kernel(const T* __restrict__ qkv, T* __
                 const float rotated = d < half ? -other : other;
                 y = y * rotation[i] + rotated * rotation[half + i];
             }
-            dst[d] = from_float<T>(y);
+            dst[d] = from_float<T>(y * factor);
         }
     }
 }
@@ -511,6 +526,114 @@ __global__ void qk_norm_rope_write_run_kernel(const __nv_bfloat16* __restrict__ 
     }
 }
 
+// The same for bfloat16 heads without norm and bias whatever the sizes of key and value heads and their numbers, in pieces of 8
+// channels: one block per RUN consecutive tokens, a thread per piece of a token's queries, keys and values in turn.  The rotation's
+// partner piece is read from the projection itself.  A run's values leave as one store per channel where they lie together.
+template <int RUN>
+__global__ void rewrite_pieces_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_pages,
+                                      __nv_bfloat16* __restrict__ v_pages, const float* __restrict__ inv_freq, int rotary_dim, const int* __restrict__ positions,
+                                      const int* __restrict__ token_segment, const int* __restrict__ block_table, PagedLayout layout, int num_heads, int write_kv,
+                                      int tokens, int* status, RewriteExtras extra) {
+    using T = __nv_bfloat16;
+    extern __shared__ float rotation[];   // per token of the run: cos[half], sin[half]
+    const int first = blockIdx.x * RUN;
+    const int count = min(RUN, tokens - first);
+    const int hd = layout.head_dim, vd = layout.value_dim, half = rotary_dim / 2;
+    const int head_pieces = hd / 8, value_pieces = vd / 8;
+    const int query_pieces = num_heads * head_pieces;
+    const int key_pieces = write_kv ? layout.num_groups * head_pieces : 0;
+    const int pieces = query_pieces + key_pieces + (write_kv ? layout.value_groups * value_pieces : 0);
+    for (int i = threadIdx.x; i < count * half; i += blockDim.x) {
+        const int t = i / half, f = i - t * half;
+        float sine, cosine;
+        sincosf(static_cast<float>(positions[first + t]) * inv_freq[f], &sine, &cosine);
+        rotation[t * rotary_dim + f] = cosine * extra.turn_scale;
+        rotation[t * rotary_dim + half + f] = sine * extra.turn_scale;
+    }
+    const int segment = token_segment[first], position0 = positions[first];
+    const bool together = RUN > 1 && count == RUN && token_segment[first + RUN - 1] == segment && positions[first + RUN - 1] == position0 + RUN - 1 &&
+                          position0 % RUN == 0 && layout.page_size % RUN == 0;
+    __syncthreads();
+    for (int piece = threadIdx.x; piece < pieces; piece += blockDim.x) {
+        const __nv_bfloat16* source = qkv + static_cast<size_t>(first) * extra.row_stride + static_cast<size_t>(piece) * 8;
+        uint4 raw[RUN];
+#pragma unroll
+        for (int t = 0; t < RUN; ++t) raw[t] = t < count ? *reinterpret_cast<const uint4*>(source + static_cast<size_t>(t) * extra.row_stride) : make_uint4(0u, 0u, 0u, 0u);
+        if (piece >= query_pieces + key_pieces) {
+            const int index = piece - query_pieces - key_pieces, group = index / value_pieces, channel = (index - group * value_pieces) * 8;
+            if constexpr (RUN == 4) {
+                if (together) {
+                    T* value = value_column(v_pages, block_table, layout, segment, position0, group);
+                    if (value == nullptr) continue;   // reported with the keys
+#pragma unroll
+                    for (int w = 0; w < 4; ++w) {
+                        const uint32_t words[4] = {(&raw[0].x)[w], (&raw[1].x)[w], (&raw[2].x)[w], (&raw[3].x)[w]};
+#pragma unroll
+                        for (int high = 0; high < 2; ++high) {
+                            const uint32_t take = high ? 0x7632 : 0x5410;
+                            *reinterpret_cast<uint2*>(value + static_cast<size_t>(channel + 2 * w + high) * layout.page_size) =
+                                make_uint2(__byte_perm(words[0], words[1], take), __byte_perm(words[2], words[3], take));
+                        }
+                    }
+                    continue;
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < RUN; ++t) {
+                if (t >= count) break;
+                T* value = value_column(v_pages, block_table, layout, token_segment[first + t], positions[first + t], group);
+                if (value == nullptr) continue;
+                const T* elements = reinterpret_cast<const T*>(&raw[t]);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) value[static_cast<size_t>(channel + i) * layout.page_size] = elements[i];
+            }
+            continue;
+        }
+        const bool is_query = piece < query_pieces;
+        const int head = piece / head_pieces, chunk = piece - head * head_pieces;   // key heads are counted on after the query heads
+        const bool rotates = chunk * 8 < rotary_dim, first_half = chunk * 8 < half;
+#pragma unroll
+        for (int t = 0; t < RUN; ++t) {
+            if (t >= count) break;
+            const int token = first + t, position = positions[token];
+            float own[8];
+            const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw[t]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 two = __bfloat1622float2(pairs[i]);
+                own[2 * i] = two.x;
+                own[2 * i + 1] = two.y;
+            }
+            if (rotates) {
+                const uint4 other_raw = *reinterpret_cast<const uint4*>(source + static_cast<size_t>(t) * extra.row_stride + (first_half ? half : -half));
+                const __nv_bfloat162* others = reinterpret_cast<const __nv_bfloat162*>(&other_raw);
+                const float* turn = rotation + t * rotary_dim + (first_half ? chunk * 8 : chunk * 8 - half);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 two = __bfloat1622float2(others[i]);
+                    own[2 * i] = own[2 * i] * turn[2 * i] + (first_half ? -two.x : two.x) * turn[half + 2 * i];
+                    own[2 * i + 1] = own[2 * i + 1] * turn[2 * i + 1] + (first_half ? -two.y : two.y) * turn[half + 2 * i + 1];
+                }
+            }
+            const float factor = is_query ? query_factor(extra, position) : 1.0f;
+            uint4 packed;
+            __nv_bfloat162* packed_pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) packed_pairs[i] = __floats2bfloat162_rn(own[2 * i] * factor, own[2 * i + 1] * factor);
+            if (is_query) {
+                *reinterpret_cast<uint4*>(q_out + (static_cast<size_t>(token) * num_heads + head) * hd + chunk * 8) = packed;
+            } else {
+                T* key_row = page_row(k_pages, block_table, layout, token_segment[token], position, head - num_heads);
+                if (key_row == nullptr) {
+                    if (chunk == 0) report_error(status, kBadPage);
+                    continue;
+                }
+                *reinterpret_cast<uint4*>(key_row + chunk * 8) = packed;
+            }
+        }
+    }
+}
+
 // grid (tokens, 2), one warp: inv[token][0] = rsqrt(mean over the q columns of x^2 + eps), inv[token][1] the same over the k columns.
 template <typename T>
 __global__ void projection_inv_rms_kernel(const T* __restrict__ qkv, int row_stride, int q_columns, int k_columns, float eps, float* __restrict__ inv) {
@@ -537,9 +660,10 @@ constexpr int kPlainMaxDimsPerThread = 4;   // head_dim <= 512
 // `keep_first` keys of its request besides (at their true positions).  Scores, softmax and the
 // weighted sum of values are 32-bit.  Keys are visited in chunks that start at key 0 (the kept
 // ones) and at the window's first key.
-template <typename T>
+// Output type TO: the activation type, or float32 for a consumer that goes on in 32-bit.
+template <typename T, typename TO>
 __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
-                                             const T* __restrict__ v_pages, T* __restrict__ out,
+                                             const T* __restrict__ v_pages, TO* __restrict__ out,
                                              const int* __restrict__ positions, const int* __restrict__ token_segment,
                                              const int* __restrict__ block_table, PagedLayout layout, int num_heads,
                                              float scale, int window, int keep_first, int* status) {
@@ -550,6 +674,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
     float* scratch = scores + kPlainChunk;       // 33
     const int token = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
     const int group = head / (num_heads / layout.num_groups);
+    const int value_group = group / (layout.num_groups / layout.value_groups);
     const int segment = token_segment[token];
     const int position = positions[token];
     const int first = window > 0 ? max(0, position - window + 1) : 0;
@@ -601,7 +726,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
                 for (int i = 0; i < count; ++i) {
                     const float p = scores[i];
                     if (p != 0.0f) {
-                        const T* v_column = value_column(const_cast<T*>(v_pages), block_table, layout, segment, chunk + i, group);
+                        const T* v_column = value_column(const_cast<T*>(v_pages), block_table, layout, segment, chunk + i, value_group);
                         if (v_column != nullptr) sum += p * to_float(v_column[static_cast<size_t>(d) * layout.page_size]);
                     }
                 }
@@ -610,13 +735,65 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
         }
         __syncthreads();   // scores[] is rewritten by the next chunk
     }
-    T* dst = out + (static_cast<size_t>(token) * num_heads + head) * vd;
+    TO* dst = out + (static_cast<size_t>(token) * num_heads + head) * vd;
     const float norm = running_sum > 0.0f ? 1.0f / running_sum : 0.0f;
 #pragma unroll
     for (int slot = 0; slot < kPlainMaxDimsPerThread; ++slot) {
         const int d = tid + slot * kPlainThreads;
-        if (d < vd) dst[d] = from_float<T>(acc[slot] * norm);
+        if (d < vd) dst[d] = from_float<TO>(acc[slot] * norm);
     }
+}
+
+// grid (tokens, slices of the heads), a warp per head; see lb_combine_maps.
+template <typename T>
+__global__ void combine_maps_kernel(const float* __restrict__ maps, const T* __restrict__ gate, int gate_stride, T* __restrict__ out, int num_heads, int num_groups,
+                                    int vd, float lambda, float eps, float factor) {
+    wait_for_previous_kernel();
+    allow_next_kernel();   // the out-projection may ask for its weights meanwhile
+    const int token = blockIdx.x, lane = threadIdx.x & 31;
+    const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (head >= num_heads) return;
+    const int per_group = num_heads / num_groups, group = head / per_group, in_group = head - group * per_group;
+    const float* a1 = maps + ((static_cast<size_t>(token) * num_groups + group) * 2 * per_group + in_group) * vd;
+    const float* a2 = a1 + static_cast<size_t>(per_group) * vd;
+    T* destination = out + (static_cast<size_t>(token) * num_heads + head) * vd;
+    const float weight = factor * (gate != nullptr ? 1.0f / (1.0f + expf(-to_float(gate[static_cast<size_t>(token) * gate_stride + head]))) : 1.0f);
+    float squares = 0.0f;
+    if (vd % 4 == 0 && vd <= 512) {
+        float4 held[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int d = 4 * lane + 128 * i;
+            held[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (d < vd) {
+                const float4 x = *reinterpret_cast<const float4*>(a1 + d), y = *reinterpret_cast<const float4*>(a2 + d);
+                held[i] = make_float4(x.x - lambda * y.x, x.y - lambda * y.y, x.z - lambda * y.z, x.w - lambda * y.w);
+            }
+            squares += held[i].x * held[i].x + held[i].y * held[i].y + held[i].z * held[i].z + held[i].w * held[i].w;
+        }
+        const float scale = rsqrtf(warp_sum(squares) / static_cast<float>(vd) + eps) * weight;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int d = 4 * lane + 128 * i;
+            if (d >= vd) break;
+            if constexpr (sizeof(T) == 2) {
+                const __nv_bfloat162 low = __floats2bfloat162_rn(held[i].x * scale, held[i].y * scale), high = __floats2bfloat162_rn(held[i].z * scale, held[i].w * scale);
+                uint2 packed;
+                packed.x = *reinterpret_cast<const uint32_t*>(&low);
+                packed.y = *reinterpret_cast<const uint32_t*>(&high);
+                *reinterpret_cast<uint2*>(destination + d) = packed;
+            } else {
+                *reinterpret_cast<float4*>(destination + d) = make_float4(held[i].x * scale, held[i].y * scale, held[i].z * scale, held[i].w * scale);
+            }
+        }
+        return;
+    }
+    for (int d = lane; d < vd; d += 32) {
+        const float o = a1[d] - lambda * a2[d];
+        squares += o * o;
+    }
+    const float scale = rsqrtf(warp_sum(squares) / static_cast<float>(vd) + eps) * weight;
+    for (int d = lane; d < vd; d += 32) destination[d] = from_float<T>((a1[d] - lambda * a2[d]) * scale);
 }
 
 }  // namespace lb
@@ -628,25 +805,29 @@ int lb_qk_norm_rope_write(const void* qkv, void* q_out, void* k_pages, void* v_p
                           const int* positions, const int* token_segment, const int* block_table, int tokens,
                           int num_heads, int num_groups, int head_dim, int page_size, int num_pages, int max_blocks,
                           int write_kv, int dtype, int* status, cudaStream_t stream, int value_dim, const float* bias, float* row_inv,
-                          float turn_scale, int row_stride) {
+                          float turn_scale, int row_stride, int value_groups, float temperature, int temperature_every) {
+    // value_groups (0: num_groups): value heads, a divisor of the key heads; temperature, temperature_every: see RewriteExtras; write_kv 0:
+    // qkv needs no more columns than the queries'.
     // row_inv: scratch [tokens][2] for a norm over the whole q and the whole k projection (null: the norm is per head);
     // turn_scale: a factor on sines and cosines; row_stride: elements between qkv's rows (0: the q, k and v columns).
     if (tokens == 0) return 0;
     if (rotary_dim < 0 || rotary_dim > head_dim || rotary_dim % 2 != 0) return -2;
     if (value_dim <= 0) value_dim = head_dim;
-    const int columns = (num_heads + num_groups) * head_dim + num_groups * value_dim;
+    if (value_groups <= 0) value_groups = num_groups;
+    if (num_groups % value_groups != 0 || temperature_every < 0) return -2;
+    const int columns = num_heads * head_dim + (write_kv ? num_groups * head_dim + value_groups * value_dim : 0);
     if (row_stride <= 0) row_stride = columns;
     if (row_stride < columns || (row_inv != nullptr && (q_weight == nullptr || bias != nullptr))) return -2;
     const int inline_whole = row_inv != nullptr && tokens <= 64 ? 1 : 0;   // the warp-per-head kernel below
-    const lb::RewriteExtras extra{row_inv, turn_scale, row_stride, inline_whole};
+    const lb::RewriteExtras extra{row_inv, turn_scale, row_stride, inline_whole, temperature, temperature_every};
     if (row_inv != nullptr && !inline_whole) {
         LB_DISPATCH_DTYPE(dtype, {
             lb::projection_inv_rms_kernel<T><<<dim3(tokens, 2), 32, 0, stream>>>(static_cast<const T*>(qkv), row_stride, num_heads * head_dim,
                                                                                  num_groups * head_dim, eps, row_inv);
         })
     }
-    lb::PagedLayout layout{page_size, num_pages, max_blocks, num_groups, head_dim, value_dim};
-    const bool plain_layout = value_dim == head_dim;   // what the 16-byte kernels below take
+    lb::PagedLayout layout{page_size, num_pages, max_blocks, num_groups, head_dim, value_dim, value_groups};
+    const bool plain_layout = value_dim == head_dim && value_groups == num_groups && temperature_every == 0;   // what the 16-byte kernels below take
     const bool power_of_two_head = head_dim == 16 || head_dim == 32 || head_dim == 64 || head_dim == 128;
     const int vector_threads = (((num_heads + num_groups) * (head_dim / 8)) + 31) / 32 * 32;
     if (tokens > 64 && plain_layout && dtype == lb::kBFloat16 && power_of_two_head && rotary_dim % 16 == 0 && rotary_dim <= head_dim && vector_threads <= 1024 &&
@@ -665,6 +846,22 @@ int lb_qk_norm_rope_write(const void* qkv, void* q_out, void* k_pages, void* v_p
             static_cast<const __nv_bfloat16*>(qkv), static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(k_pages),
             static_cast<__nv_bfloat16*>(v_pages), q_weight, k_weight, eps, scale_offset, inv_freq, rotary_dim, positions, token_segment, block_table,
             layout, num_heads, write_kv, bias, status, extra);
+        return LB_LAUNCH_RESULT();
+    }
+    if (tokens > 64 && dtype == lb::kBFloat16 && q_weight == nullptr && bias == nullptr && head_dim % 8 == 0 && value_dim % 8 == 0 && rotary_dim % 16 == 0 &&
+        row_stride % 8 == 0 &&
+        ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages)) & 15) == 0) {
+        const int pieces = (num_heads * head_dim + (write_kv ? num_groups * head_dim + value_groups * value_dim : 0)) / 8;
+        const int threads = pieces >= 256 ? 256 : (pieces + 31) / 32 * 32;
+        const size_t shared = static_cast<size_t>(rotary_dim > 0 ? rotary_dim : 2) * sizeof(float);
+        if (tokens >= lb::kRunKernelMinTokens)
+            lb::rewrite_pieces_kernel<4><<<(tokens + 3) / 4, threads, 4 * shared, stream>>>(
+                static_cast<const __nv_bfloat16*>(qkv), static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(k_pages), static_cast<__nv_bfloat16*>(v_pages),
+                inv_freq, rotary_dim, positions, token_segment, block_table, layout, num_heads, write_kv, tokens, status, extra);
+        else
+            lb::rewrite_pieces_kernel<1><<<tokens, threads, shared, stream>>>(
+                static_cast<const __nv_bfloat16*>(qkv), static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(k_pages), static_cast<__nv_bfloat16*>(v_pages),
+                inv_freq, rotary_dim, positions, token_segment, block_table, layout, num_heads, write_kv, tokens, status, extra);
         return LB_LAUNCH_RESULT();
     }
     if (tokens > 64) {
@@ -691,17 +888,40 @@ int lb_qk_norm_rope_write(const void* qkv, void* q_out, void* k_pages, void* v_p
 int lb_paged_attention_plain(const void* q, const void* k_pages, const void* v_pages, void* out, const int* positions,
                              const int* token_segment, const int* block_table, int tokens, int num_heads,
                              int num_groups, int head_dim, int page_size, int num_pages, int max_blocks, float scale,
-                             int window, int dtype, int* status, cudaStream_t stream, int value_dim, int keep_first) {
+                             int window, int dtype, int* status, cudaStream_t stream, int value_dim, int keep_first, int value_groups, int out_float) {
     if (tokens == 0) return 0;
     if (value_dim <= 0) value_dim = head_dim;
+    if (value_groups <= 0) value_groups = num_groups;
+    if (num_groups % value_groups != 0) return -2;
     if (value_dim > lb::kPlainThreads * lb::kPlainMaxDimsPerThread || num_heads % num_groups != 0 || keep_first < 0) return -2;
-    lb::PagedLayout layout{page_size, num_pages, max_blocks, num_groups, head_dim, value_dim};
+    lb::PagedLayout layout{page_size, num_pages, max_blocks, num_groups, head_dim, value_dim, value_groups};
     const dim3 grid(tokens, num_heads);
     const size_t shared = (static_cast<size_t>(head_dim) + lb::kPlainChunk + 33) * sizeof(float);
     LB_DISPATCH_DTYPE(dtype, {
-        lb::paged_attention_plain_kernel<T><<<grid, lb::kPlainThreads, shared, stream>>>(
-            static_cast<const T*>(q), static_cast<const T*>(k_pages), static_cast<const T*>(v_pages), static_cast<T*>(out),
-            positions, token_segment, block_table, layout, num_heads, scale, window, window > 0 ? keep_first : 0, status);
+        if (out_float)
+            lb::paged_attention_plain_kernel<T, float><<<grid, lb::kPlainThreads, shared, stream>>>(
+                static_cast<const T*>(q), static_cast<const T*>(k_pages), static_cast<const T*>(v_pages), static_cast<float*>(out),
+                positions, token_segment, block_table, layout, num_heads, scale, window, window > 0 ? keep_first : 0, status);
+        else
+            lb::paged_attention_plain_kernel<T, T><<<grid, lb::kPlainThreads, shared, stream>>>(
+                static_cast<const T*>(q), static_cast<const T*>(k_pages), static_cast<const T*>(v_pages), static_cast<T*>(out),
+                positions, token_segment, block_table, layout, num_heads, scale, window, window > 0 ? keep_first : 0, status);
+    })
+    return LB_LAUNCH_RESULT();
+}
+
+// The two maps of differential attention as one: per token and head,
+//   o = a1 - lambda a2;   out = T(o * rsqrt(mean(o^2) + eps) * factor * sigmoid(gate))
+// with a (float32) [tokens, groups, 2, heads_per_group, value_dim] and gate (may be null) one logit per head, `gate_stride` elements
+// from token to token; out [tokens, groups * heads_per_group * value_dim].
+int lb_combine_maps(const float* maps, const void* gate, int gate_stride, void* out, int tokens, int num_heads, int num_groups, int value_dim, float lambda, float eps,
+                    float factor, int dtype, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    if (num_groups < 1 || num_heads % num_groups != 0 || value_dim < 1) return -2;
+    const int warps = 4;
+    LB_DISPATCH_DTYPE(dtype, {
+        lb::launch_overlapped(lb::combine_maps_kernel<T>, dim3(tokens, (num_heads + warps - 1) / warps), dim3(32 * warps), 0, stream, maps, static_cast<const T*>(gate),
+                              gate_stride, static_cast<T*>(out), num_heads, num_groups, value_dim, lambda, eps, factor);
     })
     return LB_LAUNCH_RESULT();
 }

@@ -10,6 +10,8 @@
 // 16-key block so that a lane's probabilities meet contiguous bytes of the transposed value rows.
 // Every tile starts at a key index that is a multiple of 64, whatever the portion's start, so the
 // order of the sums for a token does not depend on how the prompt was cut.
+// Kernels with GENERAL = false take key and value heads of HD channels each; with GENERAL = true key heads of up to HD channels (a
+// multiple of 16) and value heads of up to HD (a multiple of 8), several key heads over one value head, and float32 output.
 #include "common.cuh"
 
 namespace lb {
@@ -47,7 +49,7 @@ struct PrefillParams {
     const __nv_bfloat16* q;         // [tokens, heads, hd]
     const __nv_bfloat16* k_pages;   // [pages, page_size, groups, hd]
     const __nv_bfloat16* v_pages;   // [pages, groups, hd, page_size]
-    __nv_bfloat16* out;             // [tokens, heads, hd]
+    void* out;                      // [tokens, heads, value_dim], bfloat16 or (out_float) float32
     const int* tiles;               // [num_tiles, 2]: first token, count
     const int* positions;
     const int* token_segment;
@@ -57,6 +59,7 @@ struct PrefillParams {
     int keep_first;   // under a window: the request's first keys that stay visible (0: none)
     float scale_log2;
     int* status;
+    int key_dim, value_dim, keys_per_value, out_float;   // GENERAL only: channels, key heads that share a value head
 };
 
 // Shared-memory pitches (bytes) that keep the fragment reads free of bank conflicts.
@@ -97,33 +100,35 @@ __device__ __forceinline__ PrefillTileEntry prefill_lookup(const PrefillParams& 
 // Copies the 64 keys of a tile into stage memory from the pages that `entry` names; blocks without a
 // page are zero-filled.  Every warp runs the loops the same number of times (the shuffles need it):
 // the counts are multiples of 32 and so is the number of threads.
-template <int HD>
+template <int HD, bool GENERAL>
 __device__ __forceinline__ void prefill_load_tile(unsigned char* stage, const PrefillParams& p, int group, PrefillTileEntry entry) {
     using Shared = PrefillShared<HD>;
-    constexpr int kChunksPerKey = HD / 8;   // 16-byte chunks in a key row
+    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
+    const int value_groups = GENERAL ? p.num_groups / p.keys_per_value : p.num_groups, value_group = GENERAL ? group / p.keys_per_value : group;
+    const int kChunksPerKey = kd / 8;   // 16-byte chunks in a key row
     unsigned char* keys = stage;
     unsigned char* values = stage + Shared::kKeyBytes;
     const int threads = blockDim.x;
-    // keys: 64 rows of HD * 2 bytes
+    // keys: 64 rows of kd * 2 bytes
     for (int index = threadIdx.x; index < kPrefillKeys * kChunksPerKey; index += threads) {
         const int row = index / kChunksPerKey, chunk = index - row * kChunksPerKey;
         const int page = __shfl_sync(0xffffffffu, entry.page, row >> 4);
         const int in_page = __shfl_sync(0xffffffffu, entry.offset, row >> 4) + (row & 15);
         void* destination = keys + row * Shared::kKeyPitch + chunk * 16;
         if (page >= 0) {
-            prefill_copy_16(destination, p.k_pages + ((static_cast<size_t>(page) * p.page_size + in_page) * p.num_groups + group) * HD + chunk * 8);
+            prefill_copy_16(destination, p.k_pages + ((static_cast<size_t>(page) * p.page_size + in_page) * p.num_groups + group) * kd + chunk * 8);
         } else {
             *reinterpret_cast<uint4*>(destination) = make_uint4(0u, 0u, 0u, 0u);
         }
     }
-    // values: HD channel rows; each 16-key block contributes two 16-byte chunks per channel
-    for (int index = threadIdx.x; index < HD * (kPrefillKeys / 8); index += threads) {
+    // values: vd channel rows; each 16-key block contributes two 16-byte chunks per channel
+    for (int index = threadIdx.x; index < vd * (kPrefillKeys / 8); index += threads) {
         const int channel = index / (kPrefillKeys / 8), chunk = index - channel * (kPrefillKeys / 8);   // chunk: 8 keys
         const int page = __shfl_sync(0xffffffffu, entry.page, chunk >> 1);
         const int in_page = __shfl_sync(0xffffffffu, entry.offset, chunk >> 1) + (chunk & 1) * 8;
         void* destination = values + channel * Shared::kValuePitch + chunk * 16;
         if (page >= 0) {
-            prefill_copy_16(destination, p.v_pages + ((static_cast<size_t>(page) * p.num_groups + group) * HD + channel) * p.page_size + in_page);
+            prefill_copy_16(destination, p.v_pages + ((static_cast<size_t>(page) * value_groups + value_group) * vd + channel) * p.page_size + in_page);
         } else {
             *reinterpret_cast<uint4*>(destination) = make_uint4(0u, 0u, 0u, 0u);
         }
@@ -134,12 +139,13 @@ __device__ __forceinline__ void prefill_load_tile(unsigned char* stage, const Pr
 // grid (num_tiles, groups * head_chunks), blockDim = 32 * heads in the chunk (<= 8 warps).
 // A tile has up to 16 * RB tokens; each warp owns RB blocks of 16 rows (tokens) of its head, which
 // share every key and value fragment read from shared memory.
-template <int HD, int RB>
+template <int HD, int RB, bool GENERAL>
 __global__ void __launch_bounds__(kPrefillMaxWarps * 32)
 attention_prefill_kernel(const PrefillParams p) {
     using Shared = PrefillShared<HD>;
     extern __shared__ __align__(16) unsigned char shared[];
     allow_next_kernel();   // the out-projection that follows may ask for its weights meanwhile
+    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
     const int heads_per_group = p.num_heads / p.num_groups;
@@ -177,8 +183,8 @@ attention_prefill_kernel(const PrefillParams p) {
             for (int half = 0; half < 2; ++half) {
                 const int row = 16 * rb + g + 8 * half;
                 uint2 loaded = make_uint2(0u, 0u);
-                if (row < count) {
-                    const __nv_bfloat16* source = p.q + (static_cast<size_t>(first_token + row) * p.num_heads + head) * HD + t * (HD / 4) + 4 * j;
+                if (row < count && (!GENERAL || 16 * j < kd)) {
+                    const __nv_bfloat16* source = p.q + (static_cast<size_t>(first_token + row) * p.num_heads + head) * kd + t * (kd / 4) + 4 * j;
                     loaded = *reinterpret_cast<const uint2*>(source);
                 }
                 q_frag[rb][j][half] = loaded.x;
@@ -204,13 +210,13 @@ attention_prefill_kernel(const PrefillParams p) {
     bool bad = false;
 
     // A tile past the list looks up nothing: its first key lies past the last position.
-    prefill_load_tile<HD>(shared, p, group, prefill_lookup(p, segment, key0_of(0), first_visible, last_position, lane, bad));
+    prefill_load_tile<HD, GENERAL>(shared, p, group, prefill_lookup(p, segment, key0_of(0), first_visible, last_position, lane, bad));
     PrefillTileEntry next_entry = prefill_lookup(p, segment, key0_of(1), first_visible, last_position, lane, bad);
     for (int tile = 0; tile < num_key_tiles; ++tile) {
         unsigned char* stage = shared + (tile & 1) * Shared::kStageBytes;
         const int key0 = key0_of(tile);
         if (tile + 1 < num_key_tiles) {
-            prefill_load_tile<HD>(shared + ((tile + 1) & 1) * Shared::kStageBytes, p, group, next_entry);
+            prefill_load_tile<HD, GENERAL>(shared + ((tile + 1) & 1) * Shared::kStageBytes, p, group, next_entry);
             next_entry = prefill_lookup(p, segment, key0_of(tile + 2), first_visible, last_position, lane, bad);
             asm volatile("cp.async.wait_group 1;\n" ::: "memory");
         } else {
@@ -224,7 +230,7 @@ attention_prefill_kernel(const PrefillParams p) {
             // does not silence a non-finite value in the product.
             const int keep_from = first_visible - key0, keep_to = last_position - key0;   // keys [from, to] of this tile are real
             const int kept_below = p.keep_first - key0;                                    // and so are the kept first keys
-            for (int index = threadIdx.x; index < HD * kPrefillKeys; index += blockDim.x) {
+            for (int index = threadIdx.x; index < vd * kPrefillKeys; index += blockDim.x) {
                 const int channel = index / kPrefillKeys, key = index - channel * kPrefillKeys;
                 if ((key < keep_from && key >= kept_below) || key > keep_to) *reinterpret_cast<__nv_bfloat16*>(values + channel * Shared::kValuePitch + key * 2) = __float2bfloat16_rn(0.0f);
             }
@@ -247,12 +253,15 @@ attention_prefill_kernel(const PrefillParams p) {
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
                     const int key = block * 16 + 4 * (g >> 1) + 2 * b + (g & 1);
-                    const unsigned char* row = stage + key * Shared::kKeyPitch + t * (HD / 4) * 2;
+                    const unsigned char* row = stage + key * Shared::kKeyPitch + t * (kd / 4) * 2;
 #pragma unroll
-                    for (int j = 0; j < HD / 16; ++j) loaded[b][j] = *reinterpret_cast<const uint2*>(row + j * 8);
+                    for (int j = 0; j < HD / 16; ++j) {
+                        if (!GENERAL || 16 * j < kd) loaded[b][j] = *reinterpret_cast<const uint2*>(row + j * 8);
+                    }
                 }
 #pragma unroll
                 for (int j = 0; j < HD / 16; ++j) {
+                    if (GENERAL && 16 * j >= kd) break;
 #pragma unroll
                     for (int b = 0; b < 2; ++b) {
 #pragma unroll
@@ -341,6 +350,7 @@ attention_prefill_kernel(const PrefillParams p) {
             if (block < blocks_here) {
 #pragma unroll
                 for (int n = 0; n < HD / 8; ++n) {
+                    if (GENERAL && 8 * n >= vd) break;
                     const uint2 loaded = *reinterpret_cast<const uint2*>(values + (8 * n + g) * Shared::kValuePitch + (block * 16 + 4 * t) * 2);
 #pragma unroll
                     for (int rb = 0; rb < RB; ++rb) mma_16816_prefill(out[rb][n], p_frag[rb][block], loaded.x, loaded.y);
@@ -362,17 +372,20 @@ attention_prefill_kernel(const PrefillParams p) {
             const int row = 16 * rb + g + 8 * half;
             if (row >= count) continue;
             const float inverse = row_sum[rb][half] > 0.0f ? 1.0f / row_sum[rb][half] : 0.0f;
-            __nv_bfloat16* destination = p.out + (static_cast<size_t>(first_token + row) * p.num_heads + head) * HD;
+            const size_t out_row = (static_cast<size_t>(first_token + row) * p.num_heads + head) * vd;
 #pragma unroll
             for (int n = 0; n < HD / 8; ++n) {
-                *reinterpret_cast<uint32_t*>(destination + 8 * n + 2 * t) =
-                    pack_bf16_prefill(out[rb][n][2 * half] * inverse, out[rb][n][2 * half + 1] * inverse);
+                if (GENERAL && 8 * n >= vd) break;
+                const float low = out[rb][n][2 * half] * inverse, high = out[rb][n][2 * half + 1] * inverse;
+                const size_t place = out_row + 8 * n + 2 * t;
+                if (GENERAL && p.out_float) *reinterpret_cast<float2*>(static_cast<float*>(p.out) + place) = make_float2(low, high);
+                else *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + place) = pack_bf16_prefill(low, high);
             }
         }
     }
 }
 
-template <int HD>
+template <int HD, bool GENERAL>
 int launch_prefill(const PrefillParams& p, int num_tiles, cudaStream_t stream) {
     using Shared = PrefillShared<HD>;
     const int heads_per_group = p.num_heads / p.num_groups;
@@ -382,7 +395,7 @@ int launch_prefill(const PrefillParams& p, int num_tiles, cudaStream_t stream) {
     const int shared = 2 * Shared::kStageBytes;
     // Two row blocks per warp (tiles of 32 tokens) while the accumulators fit the registers.
     constexpr int row_blocks = HD <= 64 ? 2 : 1;
-    auto kernel = attention_prefill_kernel<HD, row_blocks>;
+    auto kernel = attention_prefill_kernel<HD, row_blocks, GENERAL>;
     static OncePerDevice configured;
     if (allow_shared_memory(configured, kernel, shared) != cudaSuccess) return static_cast<int>(cudaGetLastError());
     kernel<<<dim3(num_tiles, p.num_groups * head_chunks, kPrefillTile / (16 * row_blocks)), warps * 32, shared, stream>>>(p);
@@ -400,14 +413,23 @@ extern "C" {
 int lb_attention_prefill(const void* q, const void* k_pages, const void* v_pages, void* out, const int* tiles, int num_tiles,
                          const int* positions, const int* token_segment, const int* block_table, int num_heads,
                          int num_groups, int head_dim, int page_size, int num_pages, int max_blocks, float scale, int window,
-                         int* status, cudaStream_t stream, int keep_first) {
+                         int* status, cudaStream_t stream, int keep_first, int value_dim, int value_groups, int out_float) {
+    // value_dim (0: head_dim), value_groups (0: num_groups) and out_float: see GENERAL above.
     if (num_tiles == 0) return 0;
+    if (value_dim <= 0) value_dim = head_dim;
+    if (value_groups <= 0) value_groups = num_groups;
+    const bool general = value_dim != head_dim || value_groups != num_groups || out_float;
+    if (general && (head_dim % 16 != 0 || head_dim < 16 || head_dim > 128 || value_dim % 8 != 0 || value_dim < 8 || value_dim > 128 || num_groups % value_groups != 0)) return -2;
     if (page_size % 16 != 0 || num_heads % num_groups != 0 || !(scale > 0.0f) || keep_first < 0) return -2;
     lb::PrefillParams p;
     p.q = static_cast<const __nv_bfloat16*>(q);
     p.k_pages = static_cast<const __nv_bfloat16*>(k_pages);
     p.v_pages = static_cast<const __nv_bfloat16*>(v_pages);
-    p.out = static_cast<__nv_bfloat16*>(out);
+    p.out = out;
+    p.key_dim = head_dim;
+    p.value_dim = value_dim;
+    p.keys_per_value = num_groups / value_groups;
+    p.out_float = out_float;
     p.tiles = tiles;
     p.positions = positions;
     p.token_segment = token_segment;
@@ -421,15 +443,22 @@ int lb_attention_prefill(const void* q, const void* k_pages, const void* v_pages
     p.keep_first = window > 0 ? keep_first : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
+    if (general) {
+        const int widest = head_dim > value_dim ? head_dim : value_dim;
+        if (widest <= 32) return lb::launch_prefill<32, true>(p, num_tiles, stream);
+        if (widest <= 64) return lb::launch_prefill<64, true>(p, num_tiles, stream);
+        if (widest <= 96) return lb::launch_prefill<96, true>(p, num_tiles, stream);
+        return lb::launch_prefill<128, true>(p, num_tiles, stream);
+    }
     switch (head_dim) {
-        case 16: return lb::launch_prefill<16>(p, num_tiles, stream);
-        case 32: return lb::launch_prefill<32>(p, num_tiles, stream);
-        case 48: return lb::launch_prefill<48>(p, num_tiles, stream);
-        case 64: return lb::launch_prefill<64>(p, num_tiles, stream);
-        case 80: return lb::launch_prefill<80>(p, num_tiles, stream);
-        case 96: return lb::launch_prefill<96>(p, num_tiles, stream);
-        case 112: return lb::launch_prefill<112>(p, num_tiles, stream);
-        case 128: return lb::launch_prefill<128>(p, num_tiles, stream);
+        case 16: return lb::launch_prefill<16, false>(p, num_tiles, stream);
+        case 32: return lb::launch_prefill<32, false>(p, num_tiles, stream);
+        case 48: return lb::launch_prefill<48, false>(p, num_tiles, stream);
+        case 64: return lb::launch_prefill<64, false>(p, num_tiles, stream);
+        case 80: return lb::launch_prefill<80, false>(p, num_tiles, stream);
+        case 96: return lb::launch_prefill<96, false>(p, num_tiles, stream);
+        case 112: return lb::launch_prefill<112, false>(p, num_tiles, stream);
+        case 128: return lb::launch_prefill<128, false>(p, num_tiles, stream);
         default: return -2;
     }
 }

@@ -17,7 +17,10 @@
 //              row of O by its sum and store it.
 // Several CTAs share an SM (64 KB of shared memory, 128 columns of tensor memory each), so that one's
 // softmax runs under another's products.  Every wait is bounded and reports through the status word.
-// Takes head size 64, pages that are multiples of 16 keys, up to 128 query heads per K/V head.
+// Takes key heads of up to 64 channels (multiples of 8, padded with zeros to 64 by the copies' out-of-bounds fill), value heads of 64 or
+// 128, pages that are multiples of 16 keys, up to 128 query heads per K/V
+// head.  Several key heads may share a value head (the maps of differential attention); the output is bfloat16 or, for a
+// consumer that goes on in 32-bit, float32.
 #include <type_traits>
 
 #include "tcgen05.cuh"
@@ -26,13 +29,15 @@ namespace lb {
 
 constexpr int kTaRows = 128;      // rows of a tile (lanes of tensor memory)
 constexpr int kTaKeys = 64;       // keys per tile
-constexpr int kTaHeadDim = 64;
+constexpr int kTaChannels = 64;    // channels of a 128-byte swizzled row
 constexpr int kTaThreads = 192;
 constexpr int kTaTileTokens = 32;  // tokens of a tile record
 constexpr float kTaMaxSlack = 8.0f;   // how far a row's maximum may outgrow its reference exponent (base 2)
 
 struct TaParams {
-    __nv_bfloat16* out;     // [tokens, heads, 64]
+    void* out;              // [tokens, heads, value_dim], bfloat16 or float32
+    int keys_per_value;     // key heads that share a value head
+    int out_float;
     const int* tiles;       // [num_tiles, 2]: first token, count <= 32
     const int* positions;
     const int* token_segment;
@@ -46,13 +51,18 @@ struct TaParams {
     int* status;
 };
 
+// VD: channels of a value head.
+template <int VD>
 struct TaShared {
-    static constexpr int kQBytes = kTaRows * kTaHeadDim * 2;           // 16 KB
+    static constexpr int kQBytes = kTaRows * kTaChannels * 2;          // 16 KB
     static constexpr int kPBytes = kTaRows * kTaKeys * 2;              // 16 KB
-    static constexpr int kKeyBytes = kTaKeys * kTaHeadDim * 2;         // 8 KB: four boxes of 16 rows
-    static constexpr int kValueBytes = kTaHeadDim * kTaKeys * 2;       // 8 KB: four boxes of 64 channels x 16 keys
+    static constexpr int kKeyBytes = kTaKeys * kTaChannels * 2;        // 8 KB: four boxes of 16 rows
+    static constexpr int kValueBox = VD * 32;                          // VD channels x 16 keys
+    static constexpr int kValueBytes = 4 * kValueBox;
     static constexpr int kStageBytes = kKeyBytes + kValueBytes;
     static constexpr int kBytes = kQBytes + kPBytes + 2 * kStageBytes + 1024 /* alignment */ + 256 /* barriers */;
+    static constexpr int kColumns = kTaKeys + VD <= 128 ? 128 : 256;   // of tensor memory: scores, output
+    static constexpr int kCtasPerSm = VD == 64 ? 3 : 2;
 };
 
 __device__ __forceinline__ void tma_load_3d(void* destination, const CUtensorMap* map, int x, int y, int z, uint64_t* barrier) {
@@ -120,16 +130,18 @@ __device__ __forceinline__ float exp2_hardware(float x) {
 }
 
 // grid (tiles, K/V heads, parts of a 32-token tile record), 192 threads.
-template <bool PAIRED>
-__global__ void __launch_bounds__(kTaThreads, 3)   // three CTAs per SM: one's softmax runs under the others' products
+template <int VD, bool PAIRED>
+__global__ void __launch_bounds__(kTaThreads, TaShared<VD>::kCtasPerSm)   // several CTAs per SM: one's softmax runs under the others' products
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                          const TaParams p) {
+    using Shared = TaShared<VD>;
+    static_assert(!PAIRED || VD == 64, "shared tiles are merged through the Q and P tiles");
     extern __shared__ unsigned char raw_shared[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(raw_shared) + 1023) & ~static_cast<uintptr_t>(1023));
     unsigned char* q_tile = base;
-    unsigned char* p_tile = base + TaShared::kQBytes;
-    unsigned char* stages = p_tile + TaShared::kPBytes;
-    uint64_t* barriers = reinterpret_cast<uint64_t*>(stages + 2 * TaShared::kStageBytes);
+    unsigned char* p_tile = base + Shared::kQBytes;
+    unsigned char* stages = p_tile + Shared::kPBytes;
+    uint64_t* barriers = reinterpret_cast<uint64_t*>(stages + 2 * Shared::kStageBytes);
     uint64_t* q_full = barriers;
     // Keys and values have barriers of their own: a stage's keys are free again as soon as S = Q K^T of
     // their tile is done, a whole softmax before its values are, and the keys of the tile after next
@@ -149,7 +161,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     allow_next_kernel();   // the out-projection that follows may ask for its weights meanwhile
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int heads_per_group = p.num_heads / p.num_groups;
-    const int group = blockIdx.y;
+    const int group = blockIdx.y, value_group = group / p.keys_per_value;
     // Tiles are listed in the order of the tokens; the last ones of a prompt see the most keys and start first.
     // With split_tiles > 0 two CTAs (a cluster) stand behind every tile record: where the tile sees many keys,
     // each takes half of them and CTA 0 merges the halves at the end (CTA 1 sends its output, exponent and sum
@@ -204,7 +216,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     if (warp == 1) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_address(tmem_slot)), "r"(128) : "memory");
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_address(tmem_slot)), "r"(Shared::kColumns) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -218,7 +230,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // table, its two boxes), so a tile costs the scheduler a quarter of the instructions one lane
         // would need; the other lanes idle along.
         if (lane == 0) {
-            barrier_expect(q_full, static_cast<uint32_t>(p.tokens_per_cta * heads_per_group * kTaHeadDim * 2));
+            barrier_expect(q_full, static_cast<uint32_t>(p.tokens_per_cta * heads_per_group * kTaChannels * 2));
             tma_load_3d(q_tile, &map_q, 0, group * heads_per_group, first_token, q_full);
         }
         bool bad = false;
@@ -245,29 +257,29 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         look_up(0, page, offset);
         for (int tile = 0; tile < num_key_tiles; ++tile) {
             const int s = tile & 1;
-            unsigned char* keys = stages + s * TaShared::kStageBytes;
-            unsigned char* values = keys + TaShared::kKeyBytes;
+            unsigned char* keys = stages + s * Shared::kStageBytes;
+            unsigned char* values = keys + Shared::kKeyBytes;
             const int this_page = page, this_offset = offset;
             look_up(tile + 1, page, offset);
-            const uint32_t bytes = 2048u * static_cast<uint32_t>(__popc(__ballot_sync(0xffffffffu, this_page >= 0)));
+            const uint32_t blocks = static_cast<uint32_t>(__popc(__ballot_sync(0xffffffffu, this_page >= 0)));
             if (tile >= 2 && !__all_sync(0xffffffffu, barrier_wait_parked(&k_free[s], ((tile >> 1) - 1) & 1))) {
                 atomicExch(&failed, 1);
                 break;
             }
-            if (lane == 0) barrier_expect(&k_full[s], bytes);
+            if (lane == 0) barrier_expect(&k_full[s], 2048u * blocks);
             if (this_page >= 0) tma_load_4d(keys + lane * 2048, &map_k, 0, group, this_offset, this_page, &k_full[s]);
             if (tile >= 2 && !__all_sync(0xffffffffu, barrier_wait_parked(&v_free[s], ((tile >> 1) - 1) & 1))) {
                 atomicExch(&failed, 1);
                 break;
             }
-            if (lane == 0) barrier_expect(&v_full[s], bytes);
-            if (this_page >= 0) tma_load_4d(values + lane * 2048, &map_v, this_offset, 0, group, this_page, &v_full[s]);
+            if (lane == 0) barrier_expect(&v_full[s], static_cast<uint32_t>(Shared::kValueBox) * blocks);
+            if (this_page >= 0) tma_load_4d(values + lane * Shared::kValueBox, &map_v, this_offset, 0, value_group, this_page, &v_full[s]);
         }
         if (__any_sync(0xffffffffu, bad) && lane == 0) report_error(p.status, kBadPage);
     } else if (warp == 1 && lane == 0) {
         // Product issuer.  It waits parked: three CTAs' issuers polling on one scheduler took the ALU
         // slots of the softmax warps there, and every tile waits for its slowest softmax warp.
-        constexpr uint32_t idesc = instruction_descriptor<kTaKeys>();   // N = 64 for both products (64 keys, 64 channels)
+        constexpr uint32_t idesc_scores = instruction_descriptor<kTaKeys>(), idesc_output = instruction_descriptor<VD>();   // N = 64 keys; VD channels
         bool ok = barrier_wait(q_full, 0);
         if (!ok) atomicExch(&failed, 1);
         const uint64_t desc_q = tile_descriptor(q_tile), desc_p = tile_descriptor(p_tile);
@@ -277,9 +289,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         auto issue_scores = [&](int tile) {
             if (!barrier_wait_parked(&k_full[tile & 1], (tile >> 1) & 1)) return false;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint64_t desc_k = tile_descriptor(stages + (tile & 1) * TaShared::kStageBytes);
+            const uint64_t desc_k = tile_descriptor(stages + (tile & 1) * Shared::kStageBytes);
 #pragma unroll
-            for (int k = 0; k < kTaHeadDim / 16; ++k) mma_f16(tmem_scores, desc_q + 2 * k, desc_k + 2 * k, idesc, k > 0);
+            for (int k = 0; k < kTaChannels / 16; ++k) mma_f16(tmem_scores, desc_q + 2 * k, desc_k + 2 * k, idesc_scores, k > 0);   // padded channels add zeros
             mma_commit(s_ready);
             mma_commit(&k_free[tile & 1]);
             return true;
@@ -290,7 +302,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         }
         for (int tile = 0; tile < num_key_tiles && ok; ++tile) {
             const int s = tile & 1;
-            unsigned char* values = stages + s * TaShared::kStageBytes + TaShared::kKeyBytes;
+            unsigned char* values = stages + s * Shared::kStageBytes + Shared::kKeyBytes;
             if (tile + 1 < num_key_tiles) {
                 if (!barrier_wait_parked(s_free, tile & 1)) {
                     atomicExch(&failed, 1);
@@ -308,7 +320,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-            for (int k = 0; k < kTaKeys / 16; ++k) mma_f16(tmem_output, desc_p + 2 * k, value_box_descriptor(values + k * 2048), idesc, tile > 0 || k > 0);
+            for (int k = 0; k < kTaKeys / 16; ++k) mma_f16(tmem_output, desc_p + 2 * k, value_box_descriptor(values + k * Shared::kValueBox), idesc_output, tile > 0 || k > 0);
             mma_commit(&v_free[s]);
             mma_commit(pv_done);
         }
@@ -385,7 +397,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 if (__any_sync(0xffffffffu, rescale != 1.0f)) {
 #pragma unroll
-                    for (int half = 0; half < 2; ++half) {
+                    for (int half = 0; half < VD / 32; ++half) {
                         uint32_t held[32];
                         tmem_load_32(tmem_output + lane_field + 32 * half, held);
 #pragma unroll
@@ -457,19 +469,20 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             if (needs_mask) {
                 // Keys outside [first visible, last position] of the tile hold whatever was left in the page,
                 // or were not loaded at all: clear their values, since a zero probability does not silence
-                // a non-finite value in the product.  64 channels x 64 keys, two threads per channel.
+                // a non-finite value in the product.  VD channels x 64 keys, 128 / VD threads per channel.
                 if (!wait_together(&v_full[s], (tile >> 1) & 1)) {
                     ok = false;
                     break;
                 }
-                unsigned char* values = stages + s * TaShared::kStageBytes + TaShared::kKeyBytes;
-                const int channel = row & 63, key_half = row >> 6;
-                for (int i = 0; i < 32; ++i) {
-                    const int local_key = 32 * key_half + i, key = key0 + local_key;
+                unsigned char* values = stages + s * Shared::kStageBytes + Shared::kKeyBytes;
+                constexpr int kKeysHere = kTaKeys * VD / kTaRows;
+                const int channel = row % VD, key_part = row / VD;
+                for (int i = 0; i < kKeysHere; ++i) {
+                    const int local_key = kKeysHere * key_part + i, key = key0 + local_key;
                     if ((key < first_visible && key >= p.keep_first) || key > last_position) {
                         const int block = local_key >> 4, in_block = local_key & 15;
                         // 32-byte swizzle: the 16-byte half of a 32-byte row is flipped in rows 4-7 of every 8
-                        unsigned char* address = values + block * 2048 + channel * 32 + ((((in_block >> 3) ^ (channel >> 2)) & 1) << 4) + (in_block & 7) * 2;
+                        unsigned char* address = values + block * Shared::kValueBox + channel * 32 + ((((in_block >> 3) ^ (channel >> 2)) & 1) << 4) + (in_block & 7) * 2;
                         *reinterpret_cast<__nv_bfloat16*>(address) = __float2bfloat16_rn(0.0f);
                     }
                 }
@@ -489,7 +502,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         float* const received_scalars = reinterpret_cast<float*>(stages);        // [128 rows][2]
         if (shared_tile) cluster_sync();
         if (shared_tile && rank == 1) {
-            const uint32_t remote_row = cluster_address(received + row * kTaHeadDim, 0);
+            const uint32_t remote_row = cluster_address(received + row * VD, 0);
             const uint32_t remote_scalars = cluster_address(received_scalars + row * 2, 0);
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
@@ -514,28 +527,35 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 row_sum = row_sum * mine + other_sum * theirs;
             }
             const float inverse = row_sum > 0.0f ? 1.0f / row_sum : 0.0f;
-            __nv_bfloat16* destination = p.out + (static_cast<size_t>(first_token + token_local) * p.num_heads + group * heads_per_group + head_local) * kTaHeadDim;
+            const size_t out_row = (static_cast<size_t>(first_token + token_local) * p.num_heads + group * heads_per_group + head_local) * VD;
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
+            for (int half = 0; half < VD / 32; ++half) {
                 uint32_t held[32];
                 tmem_load_32(tmem_output + lane_field + 32 * half, held);
                 if (valid_row && ok) {
 #pragma unroll
                     for (int chunk = 0; chunk < 4; ++chunk) {
+                        const int channel = 32 * half + 8 * chunk;
                         float values[8];
 #pragma unroll
                         for (int i = 0; i < 8; ++i) values[i] = __uint_as_float(held[8 * chunk + i]) * mine;
                         if (shared_tile) {
-                            const float4 low = *reinterpret_cast<const float4*>(received + row * kTaHeadDim + 32 * half + 8 * chunk);
-                            const float4 high = *reinterpret_cast<const float4*>(received + row * kTaHeadDim + 32 * half + 8 * chunk + 4);
+                            const float4 low = *reinterpret_cast<const float4*>(received + row * VD + 32 * half + 8 * chunk);
+                            const float4 high = *reinterpret_cast<const float4*>(received + row * VD + 32 * half + 8 * chunk + 4);
                             values[0] += low.x * theirs, values[1] += low.y * theirs, values[2] += low.z * theirs, values[3] += low.w * theirs;
                             values[4] += high.x * theirs, values[5] += high.y * theirs, values[6] += high.z * theirs, values[7] += high.w * theirs;
+                        }
+                        if (p.out_float) {
+                            float4* destination = reinterpret_cast<float4*>(static_cast<float*>(p.out) + out_row + channel);
+                            destination[0] = make_float4(values[0] * inverse, values[1] * inverse, values[2] * inverse, values[3] * inverse);
+                            destination[1] = make_float4(values[4] * inverse, values[5] * inverse, values[6] * inverse, values[7] * inverse);
+                            continue;
                         }
                         uint4 packed;
                         __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
                         for (int i = 0; i < 4; ++i) pairs[i] = __floats2bfloat162_rn(values[2 * i] * inverse, values[2 * i + 1] * inverse);
-                        *reinterpret_cast<uint4*>(destination + 32 * half + 8 * chunk) = packed;
+                        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.out) + out_row + channel) = packed;
                     }
                 }
             }
@@ -555,7 +575,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         __syncthreads();
     }
     if (warp == 1) {
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(128) : "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(Shared::kColumns) : "memory");
     }
 }
 
@@ -569,30 +589,45 @@ static bool make_paged_map(CUtensorMap* map, const void* base, int rank, const c
                   CU_TENSOR_MAP_INTERLEAVE_NONE, swizzle, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+template <int VD>
+int launch_attention_tcgen05(dim3 grid, cudaStream_t stream, const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, const TaParams& p) {
+    static OncePerDevice configured;
+    auto kernel = attention_tcgen05_kernel<VD, false>;
+    if (allow_shared_memory(configured, kernel, TaShared<VD>::kBytes) != cudaSuccess) return static_cast<int>(cudaGetLastError());
+    kernel<<<grid, kTaThreads, TaShared<VD>::kBytes, stream>>>(map_q, map_k, map_v, p);
+    return static_cast<int>(cudaGetLastError());
+}
+
 }  // namespace lb
 
 extern "C" {
 
-// Same arguments as lb_attention_prefill plus the number of tokens in q.  Returns 0, a CUDA error, -2 for
-// sizes the kernel does not take (head_dim other than 64, page_size no multiple of 16, more than 128 query
-// heads per K/V head, a scale that is not positive, pointers not 16-byte aligned), -5 if no tensor map
-// could be made.
+// Same arguments as lb_attention_prefill plus the number of tokens in q, the size of a value head (0: head_dim), the number of
+// value heads (0: num_groups; a divisor of them otherwise) and whether `out` is float32.  Returns 0, a CUDA error, -2 for
+// sizes the kernel does not take (key heads beyond 64 channels or no multiples of 8, value heads of other than 64 or 128, page_size no multiple of 16, more than 128
+// query heads per K/V head, a scale that is not positive, split tiles with heads other than 64, pointers not 16-byte aligned), -5 if no
+// tensor map could be made.
 int lb_attention_prefill_tcgen05(const void* q, const void* k_pages, const void* v_pages, void* out, const int* tiles, int num_tiles, int tokens,
                                  const int* positions, const int* token_segment, const int* block_table, int num_heads, int num_groups,
                                  int head_dim, int page_size, int num_pages, int max_blocks, float scale, int window, int split_tiles, int* status,
-                                 cudaStream_t stream, int keep_first) {
+                                 cudaStream_t stream, int keep_first, int value_dim, int value_groups, int out_float) {
     // split_tiles > 0: a pair of CTAs per tile record; a tile that sees at least that many tiles of 64 keys is
     // shared by its pair (for launches of few tiles, which the longest tile's chain of keys bounds).
     if (num_tiles == 0 || tokens == 0) return 0;
     if (split_tiles < 0 || split_tiles == 1 || keep_first < 0) return -2;
-    if (head_dim != lb::kTaHeadDim || page_size % 16 != 0 || num_groups < 1 || num_heads % num_groups != 0 || num_heads / num_groups > lb::kTaRows ||
-        !(scale > 0.0f))
+    if (value_dim <= 0) value_dim = head_dim;
+    if (value_groups <= 0) value_groups = num_groups;
+    if (head_dim < 8 || head_dim > lb::kTaChannels || head_dim % 8 != 0 || (value_dim != 64 && value_dim != 128) || page_size % 16 != 0 || num_groups < 1 ||
+        num_groups % value_groups != 0 || num_heads % num_groups != 0 || num_heads / num_groups > lb::kTaRows || !(scale > 0.0f))
         return -2;
+    if (split_tiles > 0 && (head_dim != 64 || value_dim != 64)) return -2;
     if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages) | reinterpret_cast<uintptr_t>(out)) & 15)
         return -2;
     const int heads_per_group = num_heads / num_groups;
     lb::TaParams p;
-    p.out = static_cast<__nv_bfloat16*>(out);
+    p.out = out;
+    p.keys_per_value = num_groups / value_groups;
+    p.out_float = out_float;
     p.tiles = tiles;
     p.positions = positions;
     p.token_segment = token_segment;
@@ -615,7 +650,7 @@ int lb_attention_prefill_tcgen05(const void* q, const void* k_pages, const void*
     {
         const cuuint64_t dims[3] = {static_cast<cuuint64_t>(head_dim), static_cast<cuuint64_t>(num_heads), static_cast<cuuint64_t>(tokens)};
         const cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_dim) * 2, static_cast<cuuint64_t>(num_heads) * head_dim * 2};
-        const cuuint32_t box[3] = {static_cast<cuuint32_t>(head_dim), static_cast<cuuint32_t>(heads_per_group), static_cast<cuuint32_t>(p.tokens_per_cta)};
+        const cuuint32_t box[3] = {static_cast<cuuint32_t>(lb::kTaChannels), static_cast<cuuint32_t>(heads_per_group), static_cast<cuuint32_t>(p.tokens_per_cta)};
         if (!lb::make_paged_map(&map_q, q, 3, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -5;
     }
     {
@@ -623,32 +658,31 @@ int lb_attention_prefill_tcgen05(const void* q, const void* k_pages, const void*
                                     static_cast<cuuint64_t>(num_pages)};
         const cuuint64_t strides[3] = {static_cast<cuuint64_t>(head_dim) * 2, static_cast<cuuint64_t>(num_groups) * head_dim * 2,
                                        static_cast<cuuint64_t>(page_size) * num_groups * head_dim * 2};
-        const cuuint32_t box[4] = {static_cast<cuuint32_t>(head_dim), 1, 16, 1};
+        const cuuint32_t box[4] = {static_cast<cuuint32_t>(lb::kTaChannels), 1, 16, 1};
         if (!lb::make_paged_map(&map_k, k_pages, 4, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -5;
     }
     {
-        const cuuint64_t dims[4] = {static_cast<cuuint64_t>(page_size), static_cast<cuuint64_t>(head_dim), static_cast<cuuint64_t>(num_groups),
+        const cuuint64_t dims[4] = {static_cast<cuuint64_t>(page_size), static_cast<cuuint64_t>(value_dim), static_cast<cuuint64_t>(value_groups),
                                     static_cast<cuuint64_t>(num_pages)};
-        const cuuint64_t strides[3] = {static_cast<cuuint64_t>(page_size) * 2, static_cast<cuuint64_t>(head_dim) * page_size * 2,
-                                       static_cast<cuuint64_t>(num_groups) * head_dim * page_size * 2};
-        const cuuint32_t box[4] = {16, static_cast<cuuint32_t>(head_dim), 1, 1};
+        const cuuint64_t strides[3] = {static_cast<cuuint64_t>(page_size) * 2, static_cast<cuuint64_t>(value_dim) * page_size * 2,
+                                       static_cast<cuuint64_t>(value_groups) * value_dim * page_size * 2};
+        const cuuint32_t box[4] = {16, static_cast<cuuint32_t>(value_dim), 1, 1};
         if (!lb::make_paged_map(&map_v, v_pages, 4, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_32B)) return -5;
     }
-    static lb::OncePerDevice configured, configured_paired;
-    if (lb::allow_shared_memory(configured, lb::attention_tcgen05_kernel<false>, lb::TaShared::kBytes) != cudaSuccess) return static_cast<int>(cudaGetLastError());
-    if (split_tiles > 0 && lb::allow_shared_memory(configured_paired, lb::attention_tcgen05_kernel<true>, lb::TaShared::kBytes) != cudaSuccess)
-        return static_cast<int>(cudaGetLastError());
     p.split_tiles = split_tiles;
     const unsigned parts = static_cast<unsigned>((lb::kTaTileTokens + p.tokens_per_cta - 1) / p.tokens_per_cta);
     if (split_tiles == 0) {
         const dim3 grid(num_tiles, num_groups, parts);
-        lb::attention_tcgen05_kernel<false><<<grid, lb::kTaThreads, lb::TaShared::kBytes, stream>>>(map_q, map_k, map_v, p);
-        return static_cast<int>(cudaGetLastError());
+        if (value_dim == 64) return lb::launch_attention_tcgen05<64>(grid, stream, map_q, map_k, map_v, p);
+        return lb::launch_attention_tcgen05<128>(grid, stream, map_q, map_k, map_v, p);
     }
+    static lb::OncePerDevice configured_paired;
+    if (lb::allow_shared_memory(configured_paired, lb::attention_tcgen05_kernel<64, true>, lb::TaShared<64>::kBytes) != cudaSuccess)
+        return static_cast<int>(cudaGetLastError());
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(2 * num_tiles, num_groups, parts);
     config.blockDim = dim3(lb::kTaThreads);
-    config.dynamicSmemBytes = lb::TaShared::kBytes;
+    config.dynamicSmemBytes = lb::TaShared<64>::kBytes;
     config.stream = stream;
     cudaLaunchAttribute attribute[1];
     attribute[0].id = cudaLaunchAttributeClusterDimension;
@@ -657,7 +691,7 @@ int lb_attention_prefill_tcgen05(const void* q, const void* k_pages, const void*
     attribute[0].val.clusterDim.z = 1;
     config.attrs = attribute;
     config.numAttrs = 1;
-    const cudaError_t launched = cudaLaunchKernelEx(&config, lb::attention_tcgen05_kernel<true>, map_q, map_k, map_v, p);
+    const cudaError_t launched = cudaLaunchKernelEx(&config, lb::attention_tcgen05_kernel<64, true>, map_q, map_k, map_v, p);
     if (launched != cudaSuccess) return static_cast<int>(launched);
     return static_cast<int>(cudaGetLastError());
 }

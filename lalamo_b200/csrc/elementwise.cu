@@ -451,9 +451,76 @@ __global__ void branch_norms_accumulate_kernel(float* __restrict__ residual, con
     }
 }
 
+// A polynomial of normalised powers as an activation, one block per row:
+//   out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3,   N(v) = v / sqrt(mean(v^2) + eps) over the row
+// (powers element by element), 32-bit inside, rounded once.  The row is read twice, the second time from the caches.
+template <typename T>
+__global__ void poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ coefficients, T* __restrict__ out, int dim, float eps) {
+    __shared__ float scratch[3][33];
+    wait_for_previous_kernel();
+    allow_next_kernel();
+    const T* row = z + static_cast<size_t>(blockIdx.x) * dim;
+    T* destination = out + static_cast<size_t>(blockIdx.x) * dim;
+    const bool wide = sizeof(T) == 2 && dim % 8 == 0;
+    float sums[3] = {0.0f, 0.0f, 0.0f};
+    auto count = [&](float v) {
+        const float square = v * v, cube = square * v;
+        sums[0] += square;
+        sums[1] += square * square;
+        sums[2] += cube * cube;
+    };
+    if (wide) {
+        for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(row + d);
+            const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 two = __bfloat1622float2(pairs[i]);
+                count(two.x);
+                count(two.y);
+            }
+        }
+    } else {
+        for (int d = threadIdx.x; d < dim; d += blockDim.x) count(to_float(row[d]));
+    }
+    float factor[3];
+#pragma unroll
+    for (int i = 0; i < 3; ++i) factor[i] = coefficients[i] * rsqrtf(block_sum(sums[i], scratch[i]) / static_cast<float>(dim) + eps);
+    const float constant = coefficients[3];
+    auto value = [&](float v) { return fmaf(fmaf(fmaf(factor[2], v, factor[1]), v, factor[0]), v, constant); };
+    if (wide) {
+        for (int d = 8 * threadIdx.x; d < dim; d += 8 * blockDim.x) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(row + d);
+            const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+            uint4 result;
+            __nv_bfloat162* results = reinterpret_cast<__nv_bfloat162*>(&result);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 two = __bfloat1622float2(pairs[i]);
+                results[i] = __floats2bfloat162_rn(value(two.x), value(two.y));
+            }
+            *reinterpret_cast<uint4*>(destination + d) = result;
+        }
+    } else {
+        for (int d = threadIdx.x; d < dim; d += blockDim.x) destination[d] = from_float<T>(value(to_float(row[d])));
+    }
+}
+
 }  // namespace lb
 
 extern "C" {
+
+int lb_poly_norm(const void* z, const float* coefficients, void* out, int rows, int dim, float eps, int dtype, cudaStream_t stream) {
+    if (rows == 0) return 0;
+    if (dim < 1) return -2;
+    int threads = ((dim + 7) / 8 + 31) / 32 * 32;
+    const int most = rows <= 64 ? 1024 : 256;
+    threads = threads < 64 ? 64 : (threads > most ? most : threads);
+    LB_DISPATCH_DTYPE(dtype, {
+        lb::launch_overlapped(lb::poly_norm_kernel<T>, dim3(rows), dim3(threads), 0, stream, static_cast<const T*>(z), coefficients, static_cast<T*>(out), dim, eps);
+    })
+    return LB_LAUNCH_RESULT();
+}
 
 int lb_feed_tokens(int* token_ids, const int* segment_start, const int* segment_length, const int* source, const int* sampled, int sampled_rows,
                    int segments, int* status, cudaStream_t stream) {

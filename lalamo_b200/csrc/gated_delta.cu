@@ -344,7 +344,8 @@ gdr_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const 
     }
 }
 
-// grid (tokens, slices of the heads), a warp per head: out[t, h, :] = T(o / sqrt(mean(o^2) + eps) * w * sigmoid(gate[t, h, :])).
+// grid (tokens, slices of the heads), a warp per head: out[t, h, :] = T(o / sqrt(mean(o^2) + eps) * w * sigmoid(gate[t, h, :]));
+// without gates (ag null) the last factor is left out.
 template <typename T>
 __global__ void gdr_output_kernel(const float* __restrict__ o, const T* __restrict__ ag, int ag_width, int gate_offset,
                                   const float* __restrict__ norm_weight, T* __restrict__ out, int heads, int dv, float eps, int gate_silu) {
@@ -353,15 +354,16 @@ __global__ void gdr_output_kernel(const float* __restrict__ o, const T* __restri
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     for (int head = blockIdx.y * warps + warp; head < heads; head += gridDim.y * warps) {
         const float* row = o + (static_cast<size_t>(token) * heads + head) * dv;
-        const T* gate = ag + static_cast<size_t>(token) * ag_width + gate_offset + static_cast<size_t>(head) * dv;
+        const T* gate = ag != nullptr ? ag + static_cast<size_t>(token) * ag_width + gate_offset + static_cast<size_t>(head) * dv : nullptr;
         float sum = 0.0f;
         for (int c = lane; c < dv; c += 32) sum += row[c] * row[c];
         sum = warp_sum(sum);
         const float inv = rsqrtf(sum / static_cast<float>(dv) + eps);
         T* dst = out + (static_cast<size_t>(token) * heads + head) * dv;
         for (int c = lane; c < dv; c += 32) {
-            const float z = to_float(gate[c]);
-            dst[c] = from_float<T>(row[c] * inv * norm_weight[c] * (gate_silu ? z * sigmoidf_(z) : sigmoidf_(z)));
+            const float z = gate != nullptr ? to_float(gate[c]) : 0.0f;
+            const float factor = gate == nullptr ? 1.0f : (gate_silu ? z * sigmoidf_(z) : sigmoidf_(z));
+            dst[c] = from_float<T>(row[c] * inv * norm_weight[c] * factor);
         }
     }
 }

@@ -23,7 +23,7 @@ __device__ __forceinline__ void warp_argmax(float& value, int& index) {
 // tokens: more loads on their way at once), the first warp choosing afterwards.  A logit's sum is the same either way.
 //   z[e] = x . router[e] (+ bias[e])  (32-bit);   s[e] = sigmoid(z[e])   (score_kind 0),  softmax(z)[e]   (score_kind 1)  or  z[e]  (score_kind 2)
 //   experts form `group_count` equal groups of neighbours; a group's score is the sum of its two largest s (of its
-//   only one, in groups of one); experts outside the best `group_keep` groups cannot be chosen;
+//   only one, in groups of one), or with `group_top` 1 its largest s; experts outside the best `group_keep` groups cannot be chosen;
 //   chosen[t, :] = the `top` eligible experts of largest s, in that order; weights[t, :] = their s (divided by their
 //   sum if `renormalize` is 1; the softmax over just the chosen s if it is 2), times `weight_scale`.
 //   `choice_bias` (may be null): experts (and groups) are ranked by s[e] + choice_bias[e]; the weights stay the s themselves.
@@ -34,7 +34,7 @@ template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router, int* __restrict__ chosen, float* __restrict__ weights,
                                  int tokens, int width, int experts, int top, int group_count, int group_keep, int score_kind, int renormalize,
                                  float weight_scale, int row_floats, int group_floats, const float* __restrict__ bias, int block_per_token,
-                                 const float* __restrict__ choice_bias, int extra, float* __restrict__ extra_out) {
+                                 const float* __restrict__ choice_bias, int extra, float* __restrict__ extra_out, int group_top) {
     extern __shared__ __align__(16) float shared[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int token = block_per_token ? blockIdx.x : blockIdx.x * warps + warp;
@@ -121,7 +121,7 @@ __global__ void moe_route_kernel(const T* __restrict__ x, const float* __restric
                 second = s;
             }
         }
-        group_score[group] = members >= 2 ? first + second : first;
+        group_score[group] = members >= 2 && group_top != 1 ? first + second : first;
     }
     for (int e = lane; e < experts; e += 32) candidates[e] = -INFINITY;
     __syncwarp();
@@ -565,11 +565,11 @@ extern "C" {
 
 int lb_moe_route(const void* x, const float* router, int* chosen, float* weights, int tokens, int width, int experts, int top, int group_count,
                  int group_keep, int score_kind, int renormalize, float weight_scale, int dtype, cudaStream_t stream, const float* bias,
-                 const float* choice_bias, int extra, float* extra_out) {
+                 const float* choice_bias, int extra, float* extra_out, int group_top) {
     // `router` has experts + extra rows; extra_out [tokens, extra] (see the kernel).
     if (tokens == 0) return 0;
     if (experts < 1 || top < 1 || top > experts || group_count < 1 || experts % group_count != 0 || group_keep < 1 || group_keep > group_count) return -2;
-    if (extra < 0 || (extra > 0 && extra_out == nullptr)) return -2;
+    if (extra < 0 || (extra > 0 && extra_out == nullptr) || group_top < 1 || group_top > 2) return -2;
     constexpr int kWarps = 4;
     // A warp's scratch: scores, candidates, group scores (padded so that the staged row starts on 16 bytes), and the row.
     const int scratch = (2 * experts + extra + group_count + 3) / 4 * 4;
@@ -584,7 +584,7 @@ int lb_moe_route(const void* x, const float* router, int* chosen, float* weights
         if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
         kernel<<<block_per_token ? tokens : (tokens + kWarps - 1) / kWarps, 32 * kWarps, shared, stream>>>(
             static_cast<const T*>(x), router, chosen, weights, tokens, width, experts, top, group_count, group_keep, score_kind, renormalize, weight_scale,
-            row_floats, padded_groups, bias, block_per_token, choice_bias, extra, extra_out);
+            row_floats, padded_groups, bias, block_per_token, choice_bias, extra, extra_out, group_top);
     })
     return LB_LAUNCH_RESULT();
 }

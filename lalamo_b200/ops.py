@@ -19,7 +19,7 @@ import torch
 
 from . import native
 
-__all__ = ["BiasedSum", "ExpertSum", "KernelError", "ScaledSum", "SlicedSum", "dtype_code", "launch_count", "reset_launch_count"]
+__all__ = ["BiasedSum", "ExpertSum", "KernelError", "ResidualStreams", "ScaledSum", "SlicedSum", "StreamWrite", "dtype_code", "launch_count", "reset_launch_count"]
 
 
 class KernelError(RuntimeError):
@@ -112,6 +112,29 @@ class ExpertSum:
                                      c_int(self.pair_out.shape[1]), c_int(dtype_code(self.dtype)), _stream())
         _done(code, "moe_combine")
         return out
+
+
+@dataclass
+class ResidualStreams:
+    """The residual as ``count`` parallel 32-bit streams: ``tensor`` is ``[tokens, count, width]``, or ``[tokens, width]`` while all
+    streams are still equal (before anything has been written to them)."""
+
+    tensor: torch.Tensor
+    count: int
+
+    @property
+    def equal(self) -> bool:
+        return self.tensor.dim() == 2
+
+
+@dataclass
+class StreamWrite:
+    """A sublayer's output on its way into the streams: ``X_to <- sum_from mix[from, to] X_from + write[to] output``, done by the
+    next :func:`stream_step`.  ``output`` is a tensor, a :class:`SlicedSum`, a :class:`BiasedSum` of either or an :class:`ExpertSum`."""
+
+    output: "torch.Tensor | SlicedSum | BiasedSum | ExpertSum"
+    mix: torch.Tensor  # float32 [streams, streams], indexed [from, to]
+    write: torch.Tensor  # float32 [streams]
 
 
 _ACTIVATIONS = {"silu": 0, "gelu": 1, "identity": 2, "sigmoid_limit": 3}  # the last takes a `limit`, see csrc/common.cuh
@@ -391,6 +414,142 @@ def bias_activation(x: torch.Tensor, bias: torch.Tensor | None, activation: str)
     return out
 
 
+def poly_norm(z: torch.Tensor, coefficients: torch.Tensor, eps: float) -> torch.Tensor:
+    """``c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3`` per row with ``N(v) = v / sqrt(mean(v^2) + eps)`` (32-bit inside, rounded once to
+    ``z``'s type); ``coefficients``: the four numbers in 32-bit on the device."""
+    _check(z, "z")
+    _check(coefficients, "coefficients", torch.float32)
+    if z.dim() != 2 or coefficients.numel() != 4:
+        raise KernelError("poly_norm: z must be [rows, dim] with four coefficients")
+    out = torch.empty_like(z)
+    _done(_lib().lb_poly_norm(_ptr(z), _ptr(coefficients), _ptr(out), c_int(z.shape[0]), c_int(z.shape[1]), c_float(eps), c_int(dtype_code(z.dtype)), _stream()), "poly_norm")
+    return out
+
+
+MAX_STREAMS = 8
+
+
+def stream_step(streams: ResidualStreams, update: StreamWrite | None, read: torch.Tensor, norm_weight: torch.Tensor, eps: float, dtype: torch.dtype, *,
+                keep: bool = True, rows: torch.Tensor | None = None, num_rows: int | None = None, conv: dict | None = None) -> torch.Tensor:
+    """What lies between two sublayers of a model with parallel residual streams: ``update`` written into ``streams`` (in place; ``keep=False``:
+    only worked out, not stored), ``u = sum_s read[s] X_s`` and its RMS norm ``u / sqrt(mean(u^2) + eps) * norm_weight``, all in 32-bit;
+    returns the norm in ``dtype``.  ``rows`` (its first ``num_rows`` entries): only these rows, with ``keep=False``.  ``conv``: for a step of
+    single tokens, the causal input convolution that turns ``h`` into ``h + conv(h)`` (``weight`` float32 ``[dim, taps]``, ``state``
+    ``[slots, taps - 1, dim]`` of ``dtype``, ``token_segment``, ``segment_slot``, ``status``); the state moves on."""
+    x, count = streams.tensor, streams.count
+    _check(x, "streams", torch.float32)
+    _check(read, "read", torch.float32)
+    _check(norm_weight, "norm_weight", torch.float32)
+    tokens, dim = x.shape[0], x.shape[-1]
+    if not 1 <= count <= MAX_STREAMS:
+        raise KernelError(f"stream_step: 1 to {MAX_STREAMS} streams, not {count}")
+    if (x.dim() == 3 and x.shape[1] != count) or x.dim() not in (2, 3) or read.numel() != count or norm_weight.numel() != dim:
+        raise KernelError("stream_step: streams must be [tokens, count, dim] (or [tokens, dim]), read [count], norm_weight [dim]")
+    if rows is not None and keep:
+        raise KernelError("stream_step: chosen rows are only read")
+    y = partials = bias = routed = None
+    slices = stride = 0
+    if update is not None:
+        _check(update.mix, "mix", torch.float32)
+        _check(update.write, "write", torch.float32)
+        if update.mix.shape != (count, count) or update.write.numel() != count:
+            raise KernelError("stream_step: mix must be [count, count] and write [count]")
+        output = update.output
+        if tuple(output.shape) != (tokens, dim):
+            raise KernelError("stream_step: the sublayer's output must be [tokens, dim]")
+        if isinstance(output, BiasedSum):
+            bias, output = output.bias, output.tensor
+            _check(bias, "bias", torch.float32)
+            if bias.numel() != dim:
+                raise KernelError("stream_step: a bias must have one element per column")
+        if isinstance(output, SlicedSum):
+            partials = output.partials
+            _check(partials, "partials", torch.float32)
+            if output.dtype != dtype:
+                raise KernelError("stream_step: a sliced output is rounded to the activation type")
+            slices, stride = partials.shape[0], partials.shape[1] * partials.shape[2]
+        elif isinstance(output, ExpertSum):
+            routed = output
+            for name, tensor, kind in (("pair_out", routed.pair_out, torch.float32), ("weights", routed.weights, torch.float32), ("chosen", routed.chosen, torch.int32)):
+                _check(tensor, name, kind)
+            if routed.pair_out.shape[0] != routed.chosen.numel() or routed.weights.shape != routed.chosen.shape:
+                raise KernelError("stream_step: the experts' outputs, weights and choices do not fit")
+        else:
+            y = output
+            _check(y, "output", dtype)
+    x_out = None
+    if update is not None and keep:
+        x_out = torch.empty(tokens, count, dim, dtype=torch.float32, device=x.device) if streams.equal else x
+    out_rows = tokens
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+        out_rows = rows.numel() if num_rows is None else num_rows
+        if out_rows > rows.numel():
+            raise KernelError("stream_step: fewer row indices than num_rows")
+    conv = conv or {}
+    weight, state = conv.get("weight"), conv.get("state")
+    taps = num_slots = 0
+    if weight is not None:
+        _check(weight, "conv weight", torch.float32)
+        taps = weight.shape[1]
+        if rows is not None or weight.shape[0] != dim:
+            raise KernelError("stream_step: the convolution's weight must be [dim, taps], and it runs on all rows")
+        for name in ("token_segment", "segment_slot"):
+            _check(conv[name], name, torch.int32)
+        if taps > 1:
+            _check(state, "conv state", dtype)
+            num_slots = state.shape[0]
+            if state.shape != (num_slots, taps - 1, dim):
+                raise KernelError("stream_step: the convolution's state must be [slots, taps - 1, dim]")
+    h = torch.empty(out_rows, dim, dtype=dtype, device=x.device)
+    code = _lib().lb_stream_step(_ptr(x), _ptr(x_out), c_int(1 if streams.equal else 0), c_int(count), _ptr(update.mix if update is not None else None),
+                                 _ptr(update.write if update is not None else None), _ptr(read), _ptr(y), _ptr(partials), c_int(slices), c_longlong(stride), _ptr(bias),
+                                 _ptr(routed.pair_out if routed is not None else None), _ptr(routed.weights if routed is not None else None),
+                                 _ptr(routed.chosen if routed is not None else None), c_int(routed.chosen.shape[1] if routed is not None else 0),
+                                 c_int(routed.experts if routed is not None else 0), _ptr(norm_weight), c_float(eps), _ptr(h), _ptr(rows), c_int(out_rows), c_int(dim),
+                                 _ptr(weight), _ptr(state if taps > 1 else None), _ptr(conv.get("token_segment")), _ptr(conv.get("segment_slot")), c_int(taps),
+                                 c_int(num_slots), c_int(dtype_code(dtype)), _ptr(conv.get("status")), _stream())
+    _done(code, "stream_step")
+    if x_out is not None:
+        streams.tensor = x_out
+    return h
+
+
+CONV_MAX_TAPS = 17
+
+
+def causal_conv(x: torch.Tensor, state: torch.Tensor | None, weight: torch.Tensor, *, channels: int | None = None, add_input: bool = False,
+                segment_start: torch.Tensor, segment_length: torch.Tensor, segment_slot: torch.Tensor, segments: int, max_length: int,
+                status: torch.Tensor) -> torch.Tensor:
+    """A depthwise causal convolution over each portion's tokens on the first ``channels`` columns of ``x`` (all: left out): ``y_t = sum_j
+    weight[:, j] x_(t - taps + 1 + j)``, what lies before the portion from the request's slot of ``state`` (``[slots, taps - 1, channels]``
+    in ``x``'s type), which then holds the portion's last ``taps - 1`` inputs.  ``add_input``: ``x_t + y_t`` instead.  32-bit sums,
+    rounded once.  ``max_length``: the longest portion."""
+    if not x.is_cuda or x.dim() != 2 or x.stride(1) != 1:
+        raise KernelError("causal_conv: x must be a [tokens, .] CUDA tensor with unit column stride")
+    _check(weight, "weight", torch.float32)
+    channels = x.shape[1] if channels is None else channels
+    taps = weight.shape[1]
+    if weight.shape[0] != channels or channels > x.shape[1] or not 1 <= taps <= CONV_MAX_TAPS:
+        raise KernelError(f"causal_conv: weight must be [channels, 1 to {CONV_MAX_TAPS} taps]")
+    num_slots = 0
+    if taps > 1:
+        if state is None:
+            raise KernelError("causal_conv: a convolution of more than one tap needs its state")
+        _check(state, "state", x.dtype)
+        num_slots = state.shape[0]
+        if state.shape != (num_slots, taps - 1, channels):
+            raise KernelError("causal_conv: state must be [slots, taps - 1, channels]")
+    for name, tensor in (("segment_start", segment_start), ("segment_length", segment_length), ("segment_slot", segment_slot)):
+        _check(tensor, name, torch.int32)
+    out = torch.empty(x.shape[0], channels, dtype=x.dtype, device=x.device)
+    code = _lib().lb_causal_conv(_ptr(x), c_int(x.stride(0)), _ptr(state if taps > 1 else None), _ptr(weight), _ptr(out), c_int(channels), c_int(channels), c_int(taps),
+                                 c_int(1 if add_input else 0), _ptr(segment_start), _ptr(segment_length), _ptr(segment_slot), c_int(segments), c_int(max_length),
+                                 c_int(num_slots), c_int(dtype_code(x.dtype)), _ptr(status), _stream())
+    _done(code, "causal_conv")
+    return out
+
+
 def stream_concat(stream: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float, status: torch.Tensor) -> torch.Tensor:
     """``[stream[t] | float(table[ids[t]]) * scale]`` per token, rounded to the table's type: the 32-bit residual stream and
     the embedding's output side by side, ``[tokens, 2 * dim]``."""
@@ -463,13 +622,15 @@ def gated_activation(fused: torch.Tensor, out: torch.Tensor, activation: str, li
 
 # ----------------------------------------------------------------------------- attention
 def _check_paged(k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor, num_groups: int, head_dim: int,
-                 value_dim: int | None = None) -> tuple[int, int, int]:
+                 value_dim: int | None = None, value_groups: int | None = None) -> tuple[int, int, int]:
     _check(k_pages, "k_pages")
     _check(v_pages, "v_pages", k_pages.dtype)
     _check(block_table, "block_table", torch.int32)
     if k_pages.dim() != 4 or k_pages.shape[2:] != (num_groups, head_dim):
         raise KernelError("the key cache must be [pages, page_size, groups, head_dim]")
-    if v_pages.shape != (k_pages.shape[0], num_groups, value_dim or head_dim, k_pages.shape[1]):
+    if num_groups % (value_groups or num_groups):
+        raise KernelError("the number of key heads must be a multiple of the value heads'")
+    if v_pages.shape != (k_pages.shape[0], value_groups or num_groups, value_dim or head_dim, k_pages.shape[1]):
         raise KernelError("the value cache must be [pages, groups, value_dim, page_size] (values are stored transposed)")
     if block_table.dim() != 2:
         raise KernelError("block_table must be [segments, max_blocks]")
@@ -500,19 +661,26 @@ def qk_norm_rope_write(
     bias: torch.Tensor | None = None,
     whole_norm: bool = False,
     turn_scale: float = 1.0,
+    value_groups: int | None = None,
+    temperature: float = 0.0,
+    temperature_every: int = 0,
 ) -> None:
     """Splits ``qkv`` rows into heads, applies per-head norm and rotary embedding to queries and
     keys, writes queries to ``q_out`` and keys/values into their pages.  ``value_dim``: the size of a
     value head where it differs from ``head_dim``; ``bias``: a 32-bit vector over ``qkv``'s columns,
     added before the norm.  ``whole_norm``: the norm runs over all of a token's query columns at once (and
     over all of its key columns), with weights of one element per column, in 32-bit with no rounding before the
-    rotation.  ``turn_scale`` multiplies sines and cosines.  ``qkv`` may be the first columns of a wider product."""
+    rotation.  ``turn_scale`` multiplies sines and cosines.  ``qkv`` may be the first columns of a wider product.
+    ``value_groups``: the number of value heads where several (consecutive) key heads share one.  ``temperature_every`` > 0: queries are
+    multiplied by ``1 + temperature * ln(floor((position + 1) / temperature_every) + 1)`` in 32-bit.  With ``write_kv=False`` the
+    queries' columns of ``qkv`` are all that is needed."""
     if not qkv.is_cuda or qkv.dim() != 2 or qkv.stride(1) != 1:
         raise KernelError("qk_norm_rope_write: qkv must be a [tokens, .] CUDA tensor with unit column stride")
     _check(q_out, "q_out", qkv.dtype)
     tokens = qkv.shape[0]
     value_dim = value_dim or head_dim
-    if qkv.shape[1] != (num_heads + num_groups) * head_dim + num_groups * value_dim or q_out.numel() != tokens * num_heads * head_dim:
+    needed = num_heads * head_dim + ((num_groups * head_dim + (value_groups or num_groups) * value_dim) if write_kv or bias is not None else 0)
+    if (qkv.shape[1] != needed if write_kv else qkv.shape[1] < needed) or q_out.numel() != tokens * num_heads * head_dim:
         raise KernelError("qk_norm_rope_write: qkv / q_out widths do not match the head counts")
     if whole_norm and (q_weight is None or bias is not None):
         raise KernelError("qk_norm_rope_write: a norm over the whole projection needs weights and takes no bias")
@@ -521,7 +689,7 @@ def qk_norm_rope_write(
         _check(bias, "bias", torch.float32)
         if bias.numel() != qkv.shape[1]:
             raise KernelError("qk_norm_rope_write: bias must have one element per column of qkv")
-    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim)
+    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim, value_groups)
     if k_pages.dtype != qkv.dtype:
         raise KernelError("qk_norm_rope_write: cache and activations differ in type")
     if (q_weight is None) != (k_weight is None):
@@ -543,7 +711,8 @@ def qk_norm_rope_write(
         _ptr(qkv), _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _ptr(q_weight), _ptr(k_weight), c_float(eps), c_float(scale_offset),
         _ptr(inv_freq), c_int(rotary_dim), _ptr(positions), _ptr(token_segment), _ptr(block_table), c_int(tokens), c_int(num_heads),
         c_int(num_groups), c_int(head_dim), c_int(page_size), c_int(num_pages), c_int(max_blocks), c_int(1 if write_kv else 0),
-        c_int(dtype_code(qkv.dtype)), _ptr(status), _stream(), c_int(value_dim), _ptr(bias), _ptr(row_inv), c_float(turn_scale), c_int(qkv.stride(0)))
+        c_int(dtype_code(qkv.dtype)), _ptr(status), _stream(), c_int(value_dim), _ptr(bias), _ptr(row_inv), c_float(turn_scale), c_int(qkv.stride(0)),
+        c_int(value_groups or 0), c_float(temperature), c_int(temperature_every))
     _done(code, "qk_norm_rope_write", 2 if whole_norm and tokens > 64 else 1)   # few tokens: the statistic is computed in the rewrite itself
 
 
@@ -564,17 +733,19 @@ def paged_attention_plain(
     status: torch.Tensor,
     value_dim: int | None = None,
     keep_first: int = 0,
+    value_groups: int | None = None,
 ) -> None:
     """Causal (optionally windowed) attention of every token over its request's pages.  Under a window
     the first ``keep_first`` keys of a request stay visible.  ``value_dim``: the size of a value head
-    (and of an output head) where it differs from ``head_dim``."""
+    (and of an output head) where it differs from ``head_dim``; ``value_groups``: the number of value heads where several
+    key heads share one.  ``out`` has ``q``'s type or float32."""
     _check(q, "q")
-    _check(out, "out", q.dtype)
+    _check(out, "out", out.dtype if out.dtype == torch.float32 else q.dtype)
     tokens = q.shape[0]
     value_dim = value_dim or head_dim
     if q.numel() != tokens * num_heads * head_dim or out.numel() != tokens * num_heads * value_dim:
         raise KernelError("paged_attention: q / out sizes do not match the head counts")
-    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim)
+    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim, value_groups)
     if k_pages.dtype != q.dtype:
         raise KernelError("paged_attention: cache and queries differ in type")
     if value_dim > 512:
@@ -586,8 +757,26 @@ def paged_attention_plain(
     code = _lib().lb_paged_attention_plain(
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(positions), _ptr(token_segment), _ptr(block_table), c_int(tokens),
         c_int(num_heads), c_int(num_groups), c_int(head_dim), c_int(page_size), c_int(num_pages), c_int(max_blocks), c_float(scale),
-        c_int(window if window else 0), c_int(dtype_code(q.dtype)), _ptr(status), _stream(), c_int(value_dim), c_int(keep_first))
+        c_int(window if window else 0), c_int(dtype_code(q.dtype)), _ptr(status), _stream(), c_int(value_dim), c_int(keep_first),
+        c_int(value_groups or 0), c_int(1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0))
     _done(code, "paged_attention_plain")
+
+
+def combine_maps(maps: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor, *, num_heads: int, num_groups: int, value_dim: int, lam: float, eps: float,
+                 factor: float) -> None:
+    """Differential attention's two maps as one: ``o = a1 - lam * a2`` per head, ``out = o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate)``, all
+    in 32-bit.  ``maps`` (float32) holds per token and K/V head the first map's outputs of its query heads, then the second's,
+    ``[tokens, groups, 2, heads / groups, value_dim]``; ``gate``: one logit per head, possibly a column slice of a wider product."""
+    _check(maps, "maps", torch.float32)
+    _check(out, "out")
+    tokens = out.shape[0]
+    if out.shape != (tokens, num_heads * value_dim) or maps.numel() != 2 * out.numel() or num_heads % num_groups:
+        raise KernelError("combine_maps: maps must be [tokens, groups, 2, heads / groups, value_dim] and out [tokens, heads * value_dim]")
+    if gate is not None and (not gate.is_cuda or gate.dtype != out.dtype or gate.shape != (tokens, num_heads) or gate.stride(1) != 1):
+        raise KernelError("combine_maps: gate must be [tokens, heads] of out's type with unit column stride")
+    code = _lib().lb_combine_maps(_ptr(maps), _ptr(gate), c_int(gate.stride(0) if gate is not None else 0), _ptr(out), c_int(tokens), c_int(num_heads), c_int(num_groups),
+                                  c_int(value_dim), c_float(lam), c_float(eps), c_float(factor), c_int(dtype_code(out.dtype)), _stream())
+    _done(code, "combine_maps")
 
 
 DECODE_HEAD_DIMS = (16, 32, 48, 64, 80, 96, 112, 128)
@@ -612,8 +801,10 @@ def decode_ctas_per_sm(head_dim: int) -> int:
     return _decode_ctas_per_sm[key]
 
 
-def decode_attention_supported(dtype: torch.dtype, head_dim: int, page_size: int) -> bool:
-    return dtype == torch.bfloat16 and head_dim in DECODE_HEAD_DIMS and page_size % 16 == 0
+def decode_attention_supported(dtype: torch.dtype, head_dim: int, page_size: int, value_dim: int | None = None) -> bool:
+    """``head_dim`` counts a cache row's key channels (both maps' where a row holds two)."""
+    value_dim = value_dim or head_dim
+    return dtype == torch.bfloat16 and head_dim in DECODE_HEAD_DIMS and page_size % 16 == 0 and value_dim % 8 == 0 and 8 <= value_dim <= 128
 
 
 def decode_attention_plan(tokens: int, num_heads: int, num_groups: int, max_context: int, window: int | None, head_dim: int = 64,
@@ -662,6 +853,9 @@ def attention_decode(
     num_listed: int | None = None,
     fresh_keys: int | None = None,
     keep_first: int = 0,
+    value_dim: int | None = None,
+    value_groups: int | None = None,
+    two_maps: bool = False,
 ) -> None:
     """Split-key tensor-core attention for tokens that attend alone (bfloat16 only).  Under a window the
     first ``keep_first`` keys of a request stay visible.  ``max_context``
@@ -669,10 +863,14 @@ def attention_decode(
     ``num_listed`` entries) restricts the call to some tokens of the batch.  ``fresh_keys``: the kernel
     launched just before on this stream is :func:`qk_norm_rope_write` (which lets its successor start
     early) and writes at most that many of the newest positions each token sees; the attention then
-    starts early and reads the older keys while that kernel runs.  ``None``: an ordinary launch."""
+    starts early and reads the older keys while that kernel runs.  ``None``: an ordinary launch.  ``value_dim``: the size of a value
+    head where it differs; ``value_groups``: the number of value heads where several key heads share one; ``two_maps``: a cache
+    row's keys are those of two attention maps side by side (``head_dim`` channels in all), a K/V head's query heads (of ``head_dim / 2``
+    channels) are the first map's, then the second's (``num_heads`` counts both).  ``out`` is bfloat16 or float32."""
     _check(q, "q", torch.bfloat16)
-    _check(out, "out", torch.bfloat16)
-    if q.numel() != q.shape[0] * num_heads * head_dim or out.numel() != q.numel():
+    _check(out, "out", out.dtype if out.dtype == torch.float32 else torch.bfloat16)
+    value_dim = value_dim or head_dim
+    if q.numel() != q.shape[0] * num_heads * (head_dim // 2 if two_maps else head_dim) or out.numel() != q.shape[0] * num_heads * value_dim:
         raise KernelError("attention_decode: q / out sizes do not match the head counts")
     tokens = q.shape[0]
     if token_list is not None:
@@ -680,16 +878,16 @@ def attention_decode(
         tokens = token_list.numel() if num_listed is None else num_listed
         if tokens > token_list.numel():
             raise KernelError("attention_decode: token_list is shorter than num_listed")
-    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim)
+    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim, value_groups)
     if k_pages.dtype != torch.bfloat16:
         raise KernelError("attention_decode: the cache must be bfloat16")
-    if not decode_attention_supported(q.dtype, head_dim, page_size):
+    if not decode_attention_supported(q.dtype, head_dim, page_size, value_dim):
         raise KernelError(f"attention_decode: head_dim {head_dim} (supported: {DECODE_HEAD_DIMS}) or page_size {page_size} (a multiple of 16) is not supported")
     if num_heads % num_groups:
         raise KernelError("attention_decode: num_heads must be a multiple of num_groups")
     keep_first = keep_first if window else 0
-    splits, blocks_per_split = decode_attention_plan(tokens, num_heads, num_groups, max_context, window, head_dim, keep_first=keep_first)
-    needed = tokens * num_heads * splits * (head_dim + 2)
+    splits, blocks_per_split = decode_attention_plan(tokens, num_heads, num_groups, max_context, window, max(head_dim, -(-value_dim // 16) * 16), keep_first=keep_first)
+    needed = tokens * num_heads * splits * (value_dim + 2)
     if scratch is None:
         scratch = torch.empty(needed, dtype=torch.float32, device=q.device)
     else:
@@ -700,7 +898,8 @@ def attention_decode(
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(scratch), _ptr(positions), _ptr(token_segment), _ptr(block_table),
         _ptr(token_list), c_int(tokens), c_int(num_heads), c_int(num_groups), c_int(head_dim), c_int(page_size), c_int(num_pages), c_int(max_blocks),
         c_float(scale), c_int(window if window else 0), c_int(splits), c_int(blocks_per_split), c_int(-1 if fresh_keys is None else fresh_keys),
-        _ptr(status), _stream(), c_int(keep_first))
+        _ptr(status), _stream(), c_int(keep_first), c_int(value_dim), c_int(value_groups or 0), c_int(1 if two_maps else 0),
+        c_int(1 if out.dtype == torch.float32 else 0))
     _done(code, "attention_decode", 2 if splits > 1 else 1)   # the kernel and the merge of its splits
 
 
@@ -712,6 +911,20 @@ def prefill_attention_supported(dtype: torch.dtype, num_heads: int, num_groups: 
     heads_per_group = num_heads // max(num_groups, 1)
     chunks = -(-heads_per_group // PREFILL_MAX_HEADS_PER_CTA)
     return decode_attention_supported(dtype, head_dim, page_size) and heads_per_group % chunks == 0
+
+
+def tcgen05_attention_takes(num_heads: int, num_groups: int, head_dim: int, value_dim: int, page_size: int) -> bool:
+    """Whether the tcgen05 prefill kernel takes these sizes: key heads of up to 64 channels, value heads of 64 or 128."""
+    return page_size % 16 == 0 and head_dim % 8 == 0 and 8 <= head_dim <= 64 and value_dim in (64, 128) and num_heads // max(num_groups, 1) <= 128
+
+
+def wide_prefill_attention_supported(dtype: torch.dtype, num_heads: int, num_groups: int, head_dim: int, value_dim: int, page_size: int) -> bool:
+    """Whether :func:`attention_prefill` takes key and value heads of different sizes, shared value heads and a float32 output."""
+    if dtype != torch.bfloat16:
+        return False
+    if USE_TCGEN05_ATTENTION and tcgen05_attention_takes(num_heads, num_groups, head_dim, value_dim, page_size):
+        return True
+    return value_dim % 8 == 0 and 8 <= value_dim <= 128 and prefill_attention_supported(dtype, num_heads, num_groups, head_dim, page_size)
 
 
 def attention_prefill(
@@ -734,6 +947,8 @@ def attention_prefill(
     kernel: str | None = None,
     split_tiles: int = 0,
     keep_first: int = 0,
+    value_dim: int | None = None,
+    value_groups: int | None = None,
 ) -> None:
     """Tensor-core attention for portions of prompts (bfloat16 only).  Under a window the first
     ``keep_first`` keys of a request stay visible.  ``tiles`` is ``[num_tiles, 2]``:
@@ -741,28 +956,38 @@ def attention_prefill(
     on the tcgen05 kernel (scores and output in tensor memory), the other sizes on the ``mma.sync``
     one; ``kernel="mma"`` or ``"tcgen05"`` forces one of them.  ``split_tiles`` > 1 (tcgen05 kernel only):
     a tile that sees at least that many tiles of 64 keys is worked on by two CTAs, half of the keys each,
-    for launches of few tiles that the longest tile's chain of keys would bound."""
+    for launches of few tiles that the longest tile's chain of keys would bound.  ``value_dim``: the size of a value head where it
+    differs; ``value_groups``: the number of value heads where several key heads share one; ``out`` is bfloat16 or float32.  Where one of
+    these is used the tcgen05 kernel runs if it takes the sizes (:func:`tcgen05_attention_takes`), the ``mma.sync`` one otherwise."""
     _check(q, "q", torch.bfloat16)
-    _check(out, "out", torch.bfloat16)
+    _check(out, "out", out.dtype if out.dtype == torch.float32 else torch.bfloat16)
     _check(tiles, "tiles", torch.int32)
-    if q.numel() != q.shape[0] * num_heads * head_dim or out.numel() != q.numel():
+    wide = (value_dim or head_dim) != head_dim or (value_groups or num_groups) != num_groups or out.dtype == torch.float32
+    value_dim = value_dim or head_dim
+    if q.numel() != q.shape[0] * num_heads * head_dim or out.numel() != q.shape[0] * num_heads * value_dim:
         raise KernelError("attention_prefill: q / out sizes do not match the head counts")
     if tiles.numel() < 2 * num_tiles:
         raise KernelError("attention_prefill: fewer tile records than num_tiles")
-    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim)
-    if not prefill_attention_supported(k_pages.dtype, num_heads, num_groups, head_dim, page_size):
+    page_size, num_pages, max_blocks = _check_paged(k_pages, v_pages, block_table, num_groups, head_dim, value_dim, value_groups)
+    if wide:
+        if split_tiles or not wide_prefill_attention_supported(k_pages.dtype, num_heads, num_groups, head_dim, value_dim, page_size):
+            raise KernelError(f"attention_prefill: heads of {head_dim} and {value_dim} channels over {num_groups} groups are not sizes a tensor-core kernel takes")
+        if kernel is None:
+            kernel = "tcgen05" if USE_TCGEN05_ATTENTION and tcgen05_attention_takes(num_heads, num_groups, head_dim, value_dim, page_size) else "mma"
+    elif not prefill_attention_supported(k_pages.dtype, num_heads, num_groups, head_dim, page_size):
         raise KernelError(f"attention_prefill: head_dim {head_dim} (supported: {DECODE_HEAD_DIMS}), page_size {page_size} (a multiple of 16) "
                           f"or {num_heads} heads over {num_groups} groups is not supported")
     if kernel not in (None, "mma", "tcgen05"):
         raise KernelError(f"attention_prefill: unknown kernel {kernel!r}")
-    takes_tcgen05 = head_dim == 64 and num_heads // num_groups <= 128
+    takes_tcgen05 = tcgen05_attention_takes(num_heads, num_groups, head_dim, value_dim, page_size) and (wide or head_dim == 64)
     if kernel == "tcgen05" and not takes_tcgen05:
-        raise KernelError(f"attention_prefill: the tcgen05 kernel takes head size 64 and up to 128 query heads per K/V head, not {head_dim} and {num_heads // num_groups}")
+        raise KernelError(f"attention_prefill: the tcgen05 kernel takes head size 64 (or key heads of up to 64 channels with value heads of 64 or 128) and up to 128 query heads per K/V head, not {head_dim} and {num_heads // num_groups}")
     if kernel == "tcgen05" or (kernel is None and takes_tcgen05 and USE_TCGEN05_ATTENTION):
         code = _lib().lb_attention_prefill_tcgen05(
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(tiles), c_int(num_tiles), c_int(q.shape[0]), _ptr(positions), _ptr(token_segment),
             _ptr(block_table), c_int(num_heads), c_int(num_groups), c_int(head_dim), c_int(page_size), c_int(num_pages), c_int(max_blocks),
-            c_float(scale), c_int(window if window else 0), c_int(split_tiles), _ptr(status), _stream(), c_int(keep_first if window else 0))
+            c_float(scale), c_int(window if window else 0), c_int(split_tiles), _ptr(status), _stream(), c_int(keep_first if window else 0),
+            c_int(value_dim), c_int(value_groups or 0), c_int(1 if out.dtype == torch.float32 else 0))
         if code == -5:
             raise KernelError("attention_prefill: the driver made no tensor map for these tensors")
         _done(code, "attention_prefill (tcgen05)")
@@ -770,7 +995,8 @@ def attention_prefill(
     code = _lib().lb_attention_prefill(
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(tiles), c_int(num_tiles), _ptr(positions), _ptr(token_segment), _ptr(block_table),
         c_int(num_heads), c_int(num_groups), c_int(head_dim), c_int(page_size), c_int(num_pages), c_int(max_blocks), c_float(scale),
-        c_int(window if window else 0), _ptr(status), _stream(), c_int(keep_first if window else 0))
+        c_int(window if window else 0), _ptr(status), _stream(), c_int(keep_first if window else 0), c_int(value_dim), c_int(value_groups or 0),
+        c_int(1 if out.dtype == torch.float32 else 0))
     _done(code, "attention_prefill")
 
 
@@ -1176,10 +1402,11 @@ _ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "logits": 2}
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, *, top: int, group_count: int = 1, group_keep: int = 1, score: str = "sigmoid",
               renormalize: bool = False, weight_scale: float = 1.0, bias: torch.Tensor | None = None,
-              chosen_softmax: bool = False, choice_bias: torch.Tensor | None = None, extra: int = 0) -> tuple:
+              chosen_softmax: bool = False, choice_bias: torch.Tensor | None = None, extra: int = 0,
+              group_score: str = "two_largest") -> tuple:
     """Chooses ``top`` experts per token: 32-bit router logits ``x @ router.T``, scores (``"sigmoid"`` or
     ``"softmax"``), only experts of the ``group_keep`` best of ``group_count`` groups of neighbours eligible
-    (a group's score: the sum of its two largest scores).  Returns ``(chosen int32 [tokens, top], weights
+    (a group's score: the sum of its two largest scores, or its largest with ``group_score="largest"``).  Returns ``(chosen int32 [tokens, top], weights
     float32 [tokens, top])``, the weights being the chosen scores (over their sum if ``renormalize``; their softmax
     if ``chosen_softmax``) times ``weight_scale``.  ``bias`` (32-bit, one per expert) is added to the logits;
     ``score="logits"`` ranks by the logits themselves.  ``choice_bias`` (32-bit, one per expert) is added to the scores where
@@ -1193,6 +1420,8 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, *, top: int, group_count: i
             raise KernelError("moe_route: the bias must have one element per expert")
     if score not in _ROUTER_SCORES:
         raise KernelError(f"moe_route: unknown score {score!r}; known: {sorted(_ROUTER_SCORES)}")
+    if group_score not in ("two_largest", "largest"):
+        raise KernelError(f"moe_route: unknown group score {group_score!r}; known: 'two_largest', 'largest'")
     tokens, width = x.shape
     if extra < 0 or extra >= router.shape[0]:
         raise KernelError("moe_route: the router must have rows for the experts besides the extra ones")
@@ -1212,7 +1441,8 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, *, top: int, group_count: i
     extra_out = torch.empty(tokens, extra, dtype=torch.float32, device=x.device) if extra else None
     code = _lib().lb_moe_route(_ptr(x), _ptr(router), _ptr(chosen), _ptr(weights), c_int(tokens), c_int(width), c_int(experts), c_int(top), c_int(group_count),
                                c_int(group_keep), c_int(_ROUTER_SCORES[score]), c_int(2 if chosen_softmax else 1 if renormalize else 0), c_float(weight_scale),
-                               c_int(dtype_code(x.dtype)), _stream(), _ptr(bias), _ptr(choice_bias), c_int(extra), _ptr(extra_out))
+                               c_int(dtype_code(x.dtype)), _stream(), _ptr(bias), _ptr(choice_bias), c_int(extra), _ptr(extra_out),
+                               c_int(1 if group_score == "largest" else 2))
     _done(code, "moe_route")
     if extra:
         return chosen, weights, extra_out
@@ -1331,9 +1561,9 @@ def branch_norms_accumulate(residual: torch.Tensor, terms: list, eps: float) -> 
 # ---------------------------------------------------------------------- linear attention
 def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_heads: int, key_dim: int, value_dim: int, decay_logits: torch.Tensor | None = None,
                      decay_bias: torch.Tensor | None = None, fixed_decay: torch.Tensor | None = None, tau: float = 1.0, query_scale: float = 1.0,
-                     key_scale: float = 1.0, norm_weight: torch.Tensor, norm_eps: float, gate_offset: int, gate_activation: str = "silu",
+                     key_scale: float = 1.0, norm_weight: torch.Tensor, norm_eps: float, gate_offset: int | None, gate_activation: str = "silu",
                      segment_start: torch.Tensor, segment_length: torch.Tensor, segment_slot: torch.Tensor, segments: int, status: torch.Tensor,
-                     chunk_plan: dict | None = None) -> torch.Tensor:
+                     chunk_plan: dict | None = None, lower: torch.Tensor | None = None, query_silu: bool = False) -> torch.Tensor:
     """Linear attention ``S_t = diag(a_t) S_(t-1) + k_t v_t^T; o_t = S_t^T q_t`` over the step's portions, from each request's state
     slot and back into it, then the per-head RMS norm of the read-out (times ``norm_weight``) times the gate.
 
@@ -1343,7 +1573,10 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     activation type, the bias 32-bit).  ``matrix_state`` is ``[slots, heads, key_dim, value_dim]`` in 32-bit.  Returns
     ``[tokens, heads * value_dim]`` in the activation type.  ``chunk_plan`` (see :func:`gated_delta_chunk_plan`) lets long portions run as
     chunks side by side, as the gated delta rule's do: the recurrence is linear in the state, and the chunks' further columns carry
-    their decays' products."""
+    their decays' products.
+
+    ``lower`` (32-bit, ``heads * key_dim``): the decay is ``a = lower + (1 - lower) sigmoid(decay_logits + decay_bias)`` and the key
+    ``1 - a``; ``proj`` then has no key columns (q, v).  ``query_silu``: q is silu of its columns.  ``gate_offset=None``: no gate."""
     _check(proj, "proj")
     _check(matrix_state, "matrix_state", torch.float32)
     _check(norm_weight, "norm_weight", torch.float32)
@@ -1354,13 +1587,18 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     tokens = proj.shape[0]
     if key_dim < 1 or key_dim > 256 or value_dim < 1 or num_heads < 1:
         raise KernelError(f"linear_attention: {num_heads} heads with key size {key_dim} (at most 256) and value size {value_dim} are not supported")
-    if gate_offset < 2 * num_heads * key_dim + num_heads * value_dim or proj.shape[1] < gate_offset + num_heads * value_dim:
+    columns = (1 if lower is not None else 2) * num_heads * key_dim + num_heads * value_dim
+    if proj.shape[1] < columns or (gate_offset is not None and (gate_offset < columns or proj.shape[1] < gate_offset + num_heads * value_dim)):
         raise KernelError("linear_attention: proj is too narrow for the head counts")
     num_slots = matrix_state.shape[0]
     if matrix_state.shape != (num_slots, num_heads, key_dim, value_dim) or norm_weight.numel() != value_dim:
         raise KernelError("linear_attention: matrix_state must be [slots, heads, key_dim, value_dim] and norm_weight [value_dim]")
     if (decay_logits is None) == (fixed_decay is None):
         raise KernelError("linear_attention: the decay is either fixed per head or made from logits")
+    if lower is not None:
+        _check(lower, "lower", torch.float32)
+        if decay_logits is None or lower.numel() != num_heads * key_dim:
+            raise KernelError("linear_attention: lower bounds need decay logits and heads * key_dim elements")
     if decay_logits is not None:
         if not decay_logits.is_cuda or decay_logits.dim() != 2 or decay_logits.stride(1) != 1 or decay_logits.dtype != proj.dtype or decay_logits.shape[0] != tokens \
                 or decay_logits.shape[1] < num_heads * key_dim:
@@ -1383,7 +1621,8 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     lib = _lib()
     code = lib.lb_linear_attention_prepare(_ptr(proj), c_int(proj.shape[1]), _ptr(decay_logits), c_int(decay_logits.stride(0) if decay_logits is not None else 0),
                                            _ptr(decay_bias), _ptr(fixed_decay), c_float(1.0 / tau), c_float(query_scale), c_float(key_scale), _ptr(q), _ptr(k), _ptr(v),
-                                           _ptr(decay), c_int(tokens), c_int(num_heads), c_int(key_dim), c_int(value_dim), c_int(dtype_code(proj.dtype)), _stream())
+                                           _ptr(decay), c_int(tokens), c_int(num_heads), c_int(key_dim), c_int(value_dim), c_int(dtype_code(proj.dtype)), _stream(),
+                                           _ptr(lower), c_int(1 if query_silu else 0))
     _done(code, "linear_attention_prepare")
     read_out = torch.empty(tokens, num_heads, value_dim, dtype=torch.float32, device=device)
     # the scan of the gated delta rule without its correction (no beta), long portions in chunks where that pays
@@ -1411,7 +1650,8 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
                                _ptr(status), _stream(), _ptr(direct_list), c_int(value_dim))
         _done(code, "linear_attention_scan")
     out = torch.empty(tokens, num_heads * value_dim, dtype=proj.dtype, device=device)
-    code = lib.lb_gdr_output(_ptr(read_out), _ptr(proj), c_int(proj.shape[1]), c_int(gate_offset), _ptr(norm_weight), _ptr(out), c_int(tokens),
+    gated = gate_offset is not None
+    code = lib.lb_gdr_output(_ptr(read_out), _ptr(proj if gated else None), c_int(proj.shape[1]), c_int(gate_offset if gated else 0), _ptr(norm_weight), _ptr(out), c_int(tokens),
                              c_int(num_heads), c_int(value_dim), c_float(norm_eps), c_int(dtype_code(proj.dtype)), _stream(), c_int(1 if gate_activation == "silu" else 0))
     _done(code, "linear_attention_output")
     return out
@@ -1843,6 +2083,20 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None 
     if wants_float:
         return torch.mm(x, weight.t(), out_dtype=out_dtype)
     return torch.mm(x, weight.t())
+
+
+def linear_pending(x: torch.Tensor, weight: torch.Tensor, status: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> "torch.Tensor | SlicedSum | BiasedSum":
+    """``x @ weight.T (+ bias)`` for a consumer that adds it to something: a product the kernel cuts into K slices is left as such
+    (:class:`SlicedSum`), a bias is left to be added (:class:`BiasedSum`)."""
+    _check(x, "x")
+    _check(weight, "weight", x.dtype)
+    if x.shape[-1] != weight.shape[1]:
+        raise KernelError(f"linear_pending: input width {x.shape[-1]} does not match the weight's {weight.shape[1]}")
+    if DEFER_SLICE_SUMS and USE_TCGEN05 and not skinny_supported(x, weight.shape[0]) and tcgen05_supported(x, weight.shape[0]):
+        out = linear_tcgen05(x, weight, "store", status=status, defer_sum=True)
+    else:
+        out = linear(x, weight, status=status)
+    return out if bias is None else BiasedSum(out, bias)
 
 
 def linear_bias_activation(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, activation: str,

@@ -25,6 +25,7 @@ from .. import ops
 
 __all__ = [
     "REPLAY_MAX_TOKENS",
+    "BorrowedKVNeed",
     "CacheNeed",
     "CacheView",
     "CompositeNeed",
@@ -55,7 +56,7 @@ class TensorDecl:
     ``role``: ``"matrix"`` (stored and used in the compute type), ``"vector"`` (kept in 32-bit:
     norm scales, convolution taps, biases) or ``"table"`` (integers, int32).
     ``init`` tells the random-weights mode how to fill it: ``"normal"``, ``"ones"`` (one plus
-    noise, for scales) or ``"zeros"``.
+    noise, for scales), ``"identity"`` (a square matrix: the identity plus noise) or ``"zeros"``.
     """
 
     shape: tuple[int, ...]
@@ -108,6 +109,15 @@ class PagedKVNeed(CacheNeed):
     # row b of a request lies in the page of its block table's entry b // rows at row b % rows (a page that the request holds, since
     # b // rows is no more than the block of position b * tokens_per_row)
     tokens_per_row: int = 1
+
+
+@dataclass(frozen=True)
+class BorrowedKVNeed(CacheNeed):
+    """The keys and values that the schedule entry named by ``cache_from`` holds (its one :class:`PagedKVNeed`), to be read, not written.
+    ``window`` and ``keep_first`` say how far back the borrower looks: the pages stay for as long as anyone may look at them."""
+
+    window: int | None = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -281,6 +291,9 @@ class Mixer(Part):
     # True if forward() accepts ``residual=``: it may then add its output to the 32-bit residual
     # stream itself (in the epilogue of its last product) and return ``None`` instead of the output.
     can_accumulate = False
+    # True if forward() accepts ``defer=True``: it may then return its output un-summed (an ``ops.SlicedSum``, ``ops.BiasedSum`` or
+    # ``ops.ExpertSum``) for a consumer that adds it up on its way.
+    can_defer = False
 
     def forward(self, x: torch.Tensor, step: StepInputs, cache: CacheView | None) -> torch.Tensor | None:
         raise NotImplementedError
@@ -288,6 +301,7 @@ class Mixer(Part):
 
 class FeedForward(Part):
     can_accumulate = False  # as for Mixer
+    can_defer = False
 
     def forward(self, x: torch.Tensor, step: StepInputs) -> torch.Tensor | None:
         raise NotImplementedError

@@ -19,9 +19,9 @@ from typing import Any, Callable, ClassVar, Mapping
 
 import torch
 
-from .base import CacheView, FeedForward, Mixer, Norm, Part, Runtime, StepInputs, TensorDecl, build_part, part_type
+from .base import CacheNeed, CacheView, CompositeNeed, CompositeView, FeedForward, Mixer, Norm, Part, Runtime, StepInputs, TensorDecl, build_part, part_type
 
-__all__ = ["Block", "OutputNormBlock", "PreNormBlock", "SandwichNormBlock", "block_tensor_decls", "block_type", "build_block", "register_arrangement"]
+__all__ = ["Block", "HyperBlock", "OutputNormBlock", "PreNormBlock", "SandwichNormBlock", "block_tensor_decls", "block_type", "build_block", "register_arrangement"]
 
 _ARRANGEMENTS: dict[str, type["Block"]] = {}
 
@@ -59,8 +59,8 @@ def block_tensor_decls(spec: Any) -> dict[tuple[str, str], TensorDecl]:
 
 class Block:
     """Base of the arrangements.  Building sets one attribute per role (the built part, or ``None``
-    where the specification leaves the role empty); one of the roles must be ``"mixer"``, since the
-    model asks the block's mixer what cache it needs."""
+    where the specification leaves the role empty); one of the roles must be ``"mixer"``: a block needs
+    the cache its mixer needs, unless the arrangement keeps state of its own beside it (:meth:`cache_need`)."""
 
     roles: ClassVar[tuple[str, ...]] = ()
     mixer: Mixer
@@ -75,6 +75,9 @@ class Block:
         for role, part_spec in _role_specs(spec):
             role_tensors = {local: tensor for (owner, local), tensor in tensors.items() if owner == role}
             setattr(self, role, build_part(part_spec, role_tensors, runtime))
+
+    def cache_need(self) -> CacheNeed | None:
+        return self.mixer.cache_need()
 
     def parts(self) -> list[Part]:
         return [getattr(self, role) for role in self.roles if getattr(self, role) is not None]
@@ -236,6 +239,48 @@ class SandwichNormBlock(Block):
         if ahead is not None:
             step.carry["normed_stream"] = (residual, ahead, normed)
         return None
+
+
+@register_arrangement("hyper")
+class HyperBlock(Block):
+    """A pre-norm block on parallel residual streams: ``h = norm(sum_s read[s] X_s)``, the mixer's ``h`` through a causal convolution
+    (``h + conv(h)``) where there is one, and the sublayer's output written into all streams at once.  A sublayer's write, the next
+    sublayer's read and its norm are one kernel, also across blocks: what a block returns is its last write, still to be done."""
+
+    roles = ("pre_mixer_norm", "mixer", "mixer_connection", "input_conv", "pre_ffn_norm", "ffn", "ffn_connection")
+    pre_mixer_norm: Norm
+    pre_ffn_norm: Norm | None
+    ffn: FeedForward | None
+
+    def __init__(self, spec: Any, tensors: Mapping[tuple[str, str], torch.Tensor], runtime: Runtime) -> None:
+        super().__init__(spec, tensors, runtime)
+        if (self.ffn is None) != (self.pre_ffn_norm is None) or (self.ffn is None) != (self.ffn_connection is None):
+            raise ValueError("a block on parallel streams has a feed-forward with its norm and connection, or none of the three")
+
+    def cache_need(self) -> CacheNeed | None:
+        return CompositeNeed((self.mixer.cache_need(), self.input_conv.cache_need() if self.input_conv is not None else None))
+
+    @staticmethod
+    def _run(part: "Mixer | FeedForward", h: torch.Tensor, step: StepInputs, *cache: CacheView | None):
+        from .. import ops
+
+        out = part.forward(h, step, *cache, defer=True) if part.can_defer else part.forward(h, step, *cache)
+        return out.sum() if isinstance(out, ops.ScaledSum) else out
+
+    def forward(self, residual, pending, step: StepInputs, cache: CompositeView):  # type: ignore[override]
+        """``residual``: the streams (``ops.ResidualStreams``) without ``pending`` (an ``ops.StreamWrite`` or ``None``)."""
+        from .. import ops
+
+        mixer_cache, conv_cache = cache.views
+        fused = self.input_conv.fused(step, conv_cache) if self.input_conv is not None else None
+        h = self.pre_mixer_norm.streams_forward(residual, pending, self.mixer_connection.read, conv=fused)
+        if self.input_conv is not None and fused is None:
+            h = self.input_conv.forward(h, step, conv_cache)
+        write = ops.StreamWrite(self._run(self.mixer, h, step, mixer_cache), self.mixer_connection.mix, self.mixer_connection.write)
+        if self.ffn is None:
+            return write
+        h = self.pre_ffn_norm.streams_forward(residual, write, self.ffn_connection.read)
+        return ops.StreamWrite(self._run(self.ffn, h, step), self.ffn_connection.mix, self.ffn_connection.write)
 
 
 def build_block(spec: Any, tensors: Mapping[tuple[str, str], torch.Tensor], runtime: Runtime) -> Block:

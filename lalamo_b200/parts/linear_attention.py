@@ -1,10 +1,11 @@
 """Linear attention with a decaying matrix state per head: ``S_t = diag(a_t) S_(t-1) + k_t v_t^T; o_t = S_t^T q_t``, no softmax
 and no denominator.  The decay is one fixed number per head (retention) or one number per head and key channel made from
-the token through a bottleneck, ``a = sigmoid(W_a2 (W_a1 h) + b) ** (1 / tau)`` (gated linear attention).  The read-out is
-RMS-normed per head, multiplied by an activated gate and projected out.
+the token through a bottleneck, ``a = sigmoid(W_a2 (W_a1 h) + b) ** (1 / tau)`` (gated linear attention), or it is a forget gate
+with a lower bound, ``a = l + (1 - l) sigmoid(W_f h + b)``, that also says what is written, ``k = 1 - a`` (HGRN2).  The read-out is
+RMS-normed per head, multiplied by an activated gate (if there is one) and projected out.
 
 One product gives q, k, v and the gate's logits (rows padded to a multiple of 8); the decay's logits come from two small
-products (the bottleneck padded with zeros to a multiple of 32 columns).  A kernel lays the recurrence's inputs out in 32-bit
+products (the bottleneck padded with zeros to a multiple of 32 columns), those of a forget gate from rows of the first.  A kernel lays the recurrence's inputs out in 32-bit
 with the scale on q or k and the decays; the recurrence is the scan the gated delta rule uses, without that rule's correction;
 the read-out kernel is shared with it too.  Per request the mixer holds the matrix state in 32-bit."""
 
@@ -33,20 +34,36 @@ class LinearAttention(Mixer):
     def __init__(self, spec: LinearAttentionSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         super().__init__(spec, tensors, runtime)
         heads, dk, dv = spec.num_heads, spec.key_dim, spec.value_dim
-        if spec.decay not in ("fixed", "channel"):
-            raise ValueError(f"unknown decay {spec.decay!r}; known: 'fixed', 'channel'")
-        if spec.scaled not in ("query", "key"):
-            raise ValueError(f"unknown place of the scale {spec.scaled!r}; known: 'query', 'key'")
-        if spec.gate_activation not in ("sigmoid", "silu"):
-            raise ValueError(f"unknown gate activation {spec.gate_activation!r}; known: 'sigmoid', 'silu'")
-        rows = torch.cat([tensors["q_proj"], tensors["k_proj"], tensors["v_proj"]], dim=0)
-        self.gate_offset = _round_up(rows.shape[0], 8)
-        padded = torch.zeros(_round_up(self.gate_offset + heads * dv, 8), spec.model_dim, dtype=rows.dtype)
-        padded[: rows.shape[0]] = rows
-        padded[self.gate_offset : self.gate_offset + heads * dv] = tensors["gate_proj"]
+        if spec.decay not in ("fixed", "channel", "forget"):
+            raise ValueError(f"unknown decay {spec.decay!r}; known: 'fixed', 'channel', 'forget'")
+        if spec.scaled not in ("query", "key", "none"):
+            raise ValueError(f"unknown place of the scale {spec.scaled!r}; known: 'query', 'key', 'none'")
+        if spec.gate_activation not in ("sigmoid", "silu", "none"):
+            raise ValueError(f"unknown gate activation {spec.gate_activation!r}; known: 'sigmoid', 'silu', 'none'")
+        if spec.query_activation not in ("identity", "silu"):
+            raise ValueError(f"unknown query activation {spec.query_activation!r}; known: 'identity', 'silu'")
+        # [q ; (k) ; v | gate | forget gate], each part of the product starting at a multiple of 8 rows
+        names = ["q_proj", "v_proj"] if spec.decay == "forget" else ["q_proj", "k_proj", "v_proj"]
+        parts = [torch.cat([tensors[name] for name in names], dim=0)]
+        end = _round_up(parts[0].shape[0], 8)
+        self.gate_offset = self.forget_offset = None
+        if spec.gate_activation != "none":
+            self.gate_offset, end = end, _round_up(end + heads * dv, 8)
+            parts.append(tensors["gate_proj"])
+        if spec.decay == "forget":
+            self.forget_offset, end = end, _round_up(end + heads * dk, 8)
+            parts.append(tensors["forget_proj"])
+        padded = torch.zeros(end, spec.model_dim, dtype=parts[0].dtype)
+        offset = 0
+        for part in parts:
+            padded[offset : offset + part.shape[0]] = part
+            offset = _round_up(offset + part.shape[0], 8)
         self.in_proj = runtime.matrix(padded)
-        self.fixed_decay = self.decay_down = self.decay_up = self.decay_bias = None
-        if spec.decay == "fixed":
+        self.fixed_decay = self.decay_down = self.decay_up = self.decay_bias = self.lower = None
+        if spec.decay == "forget":
+            self.decay_bias = runtime.vector(tensors["forget_bias"])
+            self.lower = runtime.vector(tensors["lower"])
+        elif spec.decay == "fixed":
             if len(spec.decay_values) != heads:
                 raise ValueError(f"{len(spec.decay_values)} fixed decays for {heads} heads")
             self.fixed_decay = runtime.vector(torch.tensor(spec.decay_values, dtype=torch.float64))
@@ -54,27 +71,34 @@ class LinearAttention(Mixer):
             if spec.decay_rank < 1 or spec.tau <= 0.0:
                 raise ValueError("a decay made from the token needs a bottleneck of positive rank and a positive tau")
             rank = _round_up(spec.decay_rank, 32)
-            down = torch.zeros(rank, spec.model_dim, dtype=rows.dtype)
+            down = torch.zeros(rank, spec.model_dim, dtype=padded.dtype)
             down[: spec.decay_rank] = tensors["decay_down"]
-            up = torch.zeros(_round_up(heads * dk, 8), rank, dtype=rows.dtype)
+            up = torch.zeros(_round_up(heads * dk, 8), rank, dtype=padded.dtype)
             up[: heads * dk, : spec.decay_rank] = tensors["decay_up"]
             self.decay_down, self.decay_up = runtime.matrix(down), runtime.matrix(up)
             self.decay_bias = runtime.vector(tensors["decay_bias"])
         self.norm_weight = runtime.vector(tensors["out_norm"] if spec.norm_weight else torch.ones(dv))
         self.out_proj = runtime.matrix(tensors["out_proj"])
         scale = dk ** -0.5
-        self.query_scale, self.key_scale = (scale, 1.0) if spec.scaled == "query" else (1.0, scale)
+        self.query_scale = scale if spec.scaled == "query" else 1.0
+        self.key_scale = scale if spec.scaled == "key" else 1.0
 
     @classmethod
     def tensor_decls(cls, spec: LinearAttentionSpec) -> dict[str, TensorDecl]:
         heads, dk, dv = spec.num_heads, spec.key_dim, spec.value_dim
         decls = {
             "q_proj": TensorDecl((heads * dk, spec.model_dim)),
-            "k_proj": TensorDecl((heads * dk, spec.model_dim)),
             "v_proj": TensorDecl((heads * dv, spec.model_dim)),
-            "gate_proj": TensorDecl((heads * dv, spec.model_dim)),
             "out_proj": TensorDecl((spec.model_dim, heads * dv)),
         }
+        if spec.decay == "forget":
+            decls["forget_proj"] = TensorDecl((heads * dk, spec.model_dim))
+            decls["forget_bias"] = TensorDecl((heads * dk,), role="vector")
+            decls["lower"] = TensorDecl((heads * dk,), role="vector", init="zeros")
+        else:
+            decls["k_proj"] = TensorDecl((heads * dk, spec.model_dim))
+        if spec.gate_activation != "none":
+            decls["gate_proj"] = TensorDecl((heads * dv, spec.model_dim))
         if spec.decay == "channel":
             decls["decay_down"] = TensorDecl((spec.decay_rank, spec.model_dim))
             decls["decay_up"] = TensorDecl((heads * dk, spec.decay_rank))
@@ -98,8 +122,10 @@ class LinearAttention(Mixer):
         return ops.gated_delta_chunk_plan(segments.start, segments.length)
 
     can_accumulate = True
+    can_defer = True
 
-    def forward(self, x: torch.Tensor, step: StepInputs, cache: SlotStateView, residual: torch.Tensor | None = None) -> torch.Tensor | None:  # type: ignore[override]
+    def forward(self, x: torch.Tensor, step: StepInputs, cache: SlotStateView, residual: torch.Tensor | None = None,  # type: ignore[override]
+                defer: bool = False) -> "torch.Tensor | ops.SlicedSum | None":
         spec = self.spec
         if not cache.owns:
             raise ValueError("a linear-attention layer cannot read another layer's state")
@@ -107,7 +133,7 @@ class LinearAttention(Mixer):
         lists, host_lists = step.plan_of(self)
         chunk_plan = dict(lists, num_chunks=host_lists["chunk_start"].size, num_long=host_lists["long_table"].size // 3, num_direct=host_lists["direct"].size)
         proj = ops.linear(x, self.in_proj, status=status)
-        logits = None
+        logits = proj[:, self.forget_offset :] if self.forget_offset is not None else None
         if self.decay_down is not None:
             logits = ops.linear(ops.linear(x, self.decay_down, status=status), self.decay_up, status=status)
         read_out = ops.linear_attention(
@@ -125,7 +151,9 @@ class LinearAttention(Mixer):
             norm_weight=self.norm_weight,
             norm_eps=spec.norm_eps,
             gate_offset=self.gate_offset,
-            gate_activation=spec.gate_activation,
+            gate_activation=spec.gate_activation if self.gate_offset is not None else "silu",
+            lower=self.lower,
+            query_silu=spec.query_activation == "silu",
             segment_start=step.segment_start,
             segment_length=step.segment_length,
             segment_slot=cache.segment_slot,
@@ -135,4 +163,6 @@ class LinearAttention(Mixer):
         )
         if residual is not None:
             return ops.linear_accumulate(read_out, self.out_proj, residual, status=status)
+        if defer:
+            return ops.linear_pending(read_out, self.out_proj, status=status)
         return ops.linear(read_out, self.out_proj, status=status)

@@ -13,7 +13,7 @@ import torch
 
 from .. import ops
 from ..config.plan import ModelPlan
-from .base import CacheNeed, CacheView, Norm, Part, Runtime, StepInputs, TensorDecl, build_part, part_type
+from .base import BorrowedKVNeed, CacheNeed, CacheView, CompositeNeed, Norm, Part, Runtime, StepInputs, TensorDecl, build_part, part_type
 from .embedding import Embedding, Head
 from .block import Block, block_tensor_decls, build_block
 
@@ -40,6 +40,13 @@ def plan_tensor_decls(plan: ModelPlan) -> dict[TensorKey, TensorDecl]:
     return decls
 
 
+def _borrows(need: CacheNeed | None) -> bool:
+    """Whether some part of the need is read from another schedule entry's cache."""
+    if isinstance(need, CompositeNeed):
+        return any(_borrows(part) for part in need.needs)
+    return isinstance(need, BorrowedKVNeed)
+
+
 class DecoderModel:
     def __init__(self, plan: ModelPlan, tensors: Mapping[TensorKey, torch.Tensor], runtime: Runtime) -> None:
         self.plan = plan
@@ -64,13 +71,15 @@ class DecoderModel:
             self.stream_mix = build_part(plan.stream_mix, mix_tensors, runtime)
         final_tensors = {local: tensor for (path, local), tensor in tensors.items() if path == ("final_norm",)}
         self.final_norm: Norm = build_part(plan.final_norm, final_tensors, runtime)  # type: ignore[assignment]
+        self.sum_of_streams = runtime.vector(torch.ones(plan.streams)) if plan.streams > 0 else None
 
     def cache_needs(self) -> list[CacheNeed | None]:
-        """For each schedule entry the cache it owns (``None``: it owns none)."""
+        """For each schedule entry the cache it needs (``None``: none of its own; an entry that borrows only keys and values says so
+        inside its need)."""
         needs: list[CacheNeed | None] = []
         for entry in self.plan.schedule:
-            need = self.blocks[entry.layer].mixer.cache_need()
-            needs.append(None if entry.cache_from is not None else need)
+            need = self.blocks[entry.layer].cache_need()
+            needs.append(need if entry.cache_from is None or _borrows(need) else None)
         return needs
 
     def step_planners(self) -> list[Part]:
@@ -114,6 +123,8 @@ class DecoderModel:
     def forward(self, step: StepInputs, caches: list[CacheView | None]) -> torch.Tensor:
         runtime = self.runtime
         residual = self.embedding.forward(step.token_ids, step.tokens, step.positions)
+        if self.plan.streams > 0:
+            residual = ops.ResidualStreams(residual, self.plan.streams)   # all streams equal: one copy is enough until something is written
         pending: torch.Tensor | None = None
         for position, entry in enumerate(self.plan.schedule):
             if entry.add_embedding:
@@ -134,5 +145,8 @@ class DecoderModel:
             pending = self.blocks[entry.layer].forward(residual, pending, step, caches[position])
         if step.wanted == 0:
             return runtime.empty(0, self.plan.vocab_size, dtype=torch.float32)
-        normed = self.final_norm.residual_forward(residual, pending, step.want_rows, step.wanted)
+        if self.sum_of_streams is not None:
+            normed = self.final_norm.streams_forward(residual, pending, self.sum_of_streams, keep=False, rows=step.want_rows, num_rows=step.wanted)
+        else:
+            normed = self.final_norm.residual_forward(residual, pending, step.want_rows, step.wanted)
         return self.head.forward(normed)

@@ -55,6 +55,14 @@ class RMSNorm(Norm):
         )
         return out
 
+    def streams_forward(self, streams: "ops.ResidualStreams", update: "ops.StreamWrite | None", read: torch.Tensor, *, keep: bool = True,
+                        rows: torch.Tensor | None = None, num_rows: int | None = None, conv: dict | None = None) -> torch.Tensor:
+        """On parallel residual streams: ``update`` written into them, then the norm of ``sum_s read[s] X_s``, one kernel
+        (``ops.stream_step``; an exact norm without a scale offset)."""
+        if not self.spec.exact or self.spec.scale_offset != 0.0:
+            raise ValueError("parallel streams are read through an exact RMS norm with a plain weight")
+        return ops.stream_step(streams, update, read, self.scale, self.spec.eps, self.runtime.dtype, keep=keep, rows=rows, num_rows=num_rows, conv=conv)
+
     def accumulate(self, residual: torch.Tensor, delta: "torch.Tensor | ops.ScaledSum", rounded: torch.Tensor | None = None,
                    then: "RMSNorm | None" = None) -> None:
         """``residual += norm(delta)`` on the 32-bit stream, the norm itself in 32-bit too (no rounding of the

@@ -1,7 +1,8 @@
 """Rotary position embedding (``lalamo/modules/rope.py:94-102``): the inverse frequencies
 ``theta ** (-2i / rotary_dim)`` as a 32-bit table; angles, sines and cosines are computed
 in 32-bit inside the kernel that applies them.  With a :class:`~lalamo_b200.config.plan.YarnScaling` the
-table holds the stretched frequencies and ``magnitude`` the factor on sines and cosines."""
+table holds the stretched frequencies and ``magnitude`` the factor on sines and cosines; with a
+:class:`~lalamo_b200.config.plan.LlamaScaling` it holds the frequencies that rule slows down."""
 
 from __future__ import annotations
 
@@ -10,10 +11,10 @@ from typing import Mapping
 
 import torch
 
-from ..config.plan import RopeSpec, YarnScaling
+from ..config.plan import LlamaScaling, RopeSpec, YarnScaling
 from .base import PositionEncoding, Runtime, register_part
 
-__all__ = ["Rope", "stretched_frequencies"]
+__all__ = ["Rope", "slowed_frequencies", "stretched_frequencies"]
 
 
 def stretched_frequencies(rotary_dim: int, theta: float, scaling: YarnScaling) -> tuple[torch.Tensor, float]:
@@ -34,6 +35,19 @@ def stretched_frequencies(rotary_dim: int, theta: float, scaling: YarnScaling) -
     return blended.to(torch.float32), 0.1 * math.log(scaling.factor) + 1.0
 
 
+def slowed_frequencies(rotary_dim: int, theta: float, scaling: LlamaScaling) -> torch.Tensor:
+    """The frequencies ``[rotary_dim / 2]`` in 32-bit under ``scaling``, worked out in 64-bit: fast pairs as they are, slow ones divided by
+    ``factor``, blended in between by the original context's length in wavelengths."""
+    index = torch.arange(rotary_dim // 2, dtype=torch.float64)
+    frequency = torch.tensor(float(theta), dtype=torch.float64) ** (-2.0 * index / rotary_dim)
+    wavelength = 2.0 * math.pi / frequency
+    span = scaling.high - scaling.low
+    share = (scaling.original / wavelength - scaling.low) / (span if span != 0.0 else 1.0)
+    blended = (1.0 - share) * frequency / scaling.factor + share * frequency
+    slowed = torch.where(wavelength > scaling.original / scaling.low, frequency / scaling.factor, blended)
+    return torch.where(wavelength < scaling.original / scaling.high, frequency, slowed).to(torch.float32)
+
+
 @register_part(RopeSpec)
 class Rope(PositionEncoding):
     def __init__(self, spec: RopeSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
@@ -44,6 +58,8 @@ class Rope(PositionEncoding):
         if spec.scaling is None:
             channel = torch.arange(0, spec.rotary_dim, 2, dtype=torch.float32)
             inverse = 1.0 / (torch.tensor(spec.theta, dtype=torch.float32) ** (channel / spec.rotary_dim))
+        elif isinstance(spec.scaling, LlamaScaling):
+            inverse = slowed_frequencies(spec.rotary_dim, spec.theta, spec.scaling)
         else:
             inverse, self.magnitude = stretched_frequencies(spec.rotary_dim, spec.theta, spec.scaling)
         self.rotary_dim = spec.rotary_dim

@@ -63,20 +63,22 @@ class RoutedMLP(FeedForward):
         return [self.shared] if self.shared is not None else []
 
     can_accumulate = True
+    can_defer = True
 
-    def forward(self, x: torch.Tensor, step: StepInputs | None = None, residual: torch.Tensor | None = None) -> "torch.Tensor | ops.ScaledSum | None":
+    def forward(self, x: torch.Tensor, step: StepInputs | None = None, residual: torch.Tensor | None = None, defer: bool = False) -> "torch.Tensor | ops.ScaledSum | ops.ExpertSum | None":
         """The experts' weighted sum; with a shared feed-forward the two terms are handed on un-summed
         (``ops.ScaledSum``), for a consumer that adds them in 32-bit.  With ``residual`` (the 32-bit stream) everything is
-        added to it by one kernel, nothing rounded on the way, and ``None`` is returned."""
+        added to it by one kernel, nothing rounded on the way, and ``None`` is returned.  ``defer``: without a shared
+        feed-forward the weighted sum is left to the consumer (``ops.ExpertSum``)."""
         spec = self.spec
         routing = ops.moe_route(x, self.router, top=spec.top, group_count=spec.group_count, group_keep=spec.group_keep, score=spec.score,
                                 renormalize=spec.renormalize, bias=self.router_bias, chosen_softmax=spec.chosen_softmax, weight_scale=spec.weight_scale,
-                                choice_bias=self.choice_bias, extra=1 if spec.shared_gate else 0)
+                                choice_bias=self.choice_bias, extra=1 if spec.shared_gate else 0, group_score=spec.group_score)
         chosen, weights = routing[0], routing[1]
         shared_gate = routing[2] if spec.shared_gate else None
         # with a shared feed-forward the consumer adds two terms anyway: the experts' weighted sum is left to it as well
         routed = ops.moe_experts(x, self.gate, self.up, self.down, chosen, weights, spec.activation, limit=spec.limit,
-                                 combine=self.shared is None and residual is None)
+                                 combine=self.shared is None and residual is None and not defer)
         everyone = None
         if self.shared is not None:
             everyone = self.shared.forward(x, step)

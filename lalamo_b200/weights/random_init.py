@@ -43,6 +43,8 @@ def random_tensors(config: ArchitectureConfig, seed: int, std: float = 0.02, dty
             values = torch.randn(decl.shape, generator=generator, dtype=torch.float32) * std
             if decl.init == "ones":
                 values += 1.0
+            elif decl.init == "identity":
+                values += torch.eye(*decl.shape)
         storage = torch.float32 if decl.role == "vector" else _DTYPES[dtype]
         shape = shape_hook(path, local, decl.shape) if shape_hook else decl.shape
         tensors[name] = values.to(storage).reshape(shape)
