@@ -199,8 +199,8 @@ class Attention(Mixer):
             paged: CacheNeed = BorrowedKVNeed(window=spec.window, keep_first=self.keep_first)
         else:
             # a row of the cache holds both maps' keys of a K/V head side by side
-            paged = PagedKVNeed(num_groups=spec.num_groups, head_dim=self.maps * spec.head_dim, window=spec.window,
-                                value_dim=spec.value_dim if self.maps == 1 else self.value_dim, keep_first=self.keep_first)
+            paged = PagedKVNeed(num_groups=spec.num_groups, head_dim=spec.head_dim * (2 if spec.differential is not None else 1), window=spec.window,
+                                value_dim=spec.value_dim if spec.differential is None else self.value_dim, keep_first=self.keep_first)
         if spec.conv_taps > 1:
             return CompositeNeed((paged, SlotStateNeed(shape=(spec.conv_taps - 1, self.qkv_width))))
         return paged
