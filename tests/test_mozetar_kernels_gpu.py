@@ -183,7 +183,8 @@ def test_forget_recurrence(dtype):
         weight, state = 1.0 + 0.1 * torch.randn(dv, generator=generator), torch.randn(5, heads, dk, dv, generator=generator)
         slots, starts = [3, 0, 4], np.cumsum([0] + lengths[:-1]).tolist()
         device_state, device_proj, status = on(state), on(proj, dtype), zero_status()
-        plan = {name: ints(array.tolist()) for name, array in (host := ops.gated_delta_chunk_plan(starts, lengths)).items()}
+        host = ops.gated_delta_chunk_plan(starts, lengths)
+        plan = {name: ints(array.tolist()) for name, array in host.items()}
         plan.update(num_chunks=host["chunk_start"].size, num_long=host["long_table"].size // 3, num_direct=host["direct"].size)
         out = ops.linear_attention(device_proj, device_state, num_heads=heads, key_dim=dk, value_dim=dv, decay_logits=device_proj[:, start_f:], decay_bias=on(bias),
                                    lower=on(lower), query_silu=True, norm_weight=on(weight), norm_eps=1e-5, gate_offset=None, segment_start=ints(starts),
@@ -245,13 +246,12 @@ def attention_case(dtype, heads, groups, kd, vd, value_groups, window, contexts,
             k_pages[page, row], v_pages[page, :, :, row] = k[position], v[position]
         each = groups // value_groups
         want = torch.zeros(length, heads, vd, dtype=torch.float64)
-        for n in range(length):
-            i = context + n
-            first = 0 if window is None else max(0, i - window + 1)
-            for head in range(heads):
-                g = head // (heads // groups)
-                weight = torch.softmax(k[first : i + 1, g].double() @ q[n, head].double() * kd**-0.5, dim=0)
-                want[n, head] = weight @ v[first : i + 1, g // each].double()
+        i, j = torch.arange(context, total)[:, None], torch.arange(total)[None]
+        seen = (j <= i) if window is None else (j <= i) & (i - j < window)
+        for head in range(heads):
+            g = head // (heads // groups)
+            score = q[:, head].double() @ k[:, g].double().T * kd**-0.5
+            want[:, head] = torch.softmax(score.masked_fill(~seen, float("-inf")), dim=1) @ v[:, g // each].double()
         queries.append(q.reshape(length, heads * kd))
         wants.append(want.reshape(length, heads * vd))
     tokens = sum(lengths)

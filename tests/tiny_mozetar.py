@@ -143,9 +143,8 @@ def tensor_shapes(config: dict) -> dict[str, tuple[int, ...]]:
     return shapes
 
 
-def random_weights(config: dict, seed: int, sharp: bool = False) -> dict[str, torch.Tensor]:
-    """bfloat16 tensors: matrices N(0, 1/in); norm weights around one; queries and keys whose scores spread (``sharp``: over tens of
-    units, so that single keys decide); forget gates that forget over tens of tokens above lower bounds between zero and a half;
+def random_weights(config: dict, seed: int) -> dict[str, torch.Tensor]:
+    """bfloat16 tensors: matrices N(0, 1/in); norm weights around one; queries and keys whose scores spread; forget gates that forget over tens of tokens above lower bounds between zero and a half;
     streams read and written with unequal weights of either sign, mixing matrices near the identity."""
     generator = np.random.default_rng(seed)
     tensors: dict[str, torch.Tensor] = {}
@@ -155,7 +154,7 @@ def random_weights(config: dict, seed: int, sharp: bool = False) -> dict[str, to
         if last in ("norm", "norm1", "norm2"):
             values = 1.0 + 0.2 * normal
         elif ".hc" in name:
-            values = np.eye(shape[0]) + 0.2 * normal if last == "mix" else (1.0 if last == "out" else 1.0 / shape[0]) + 0.4 * normal
+            values = np.eye(shape[0]) + 0.2 * normal if last == "mix" else (1.0 if last == "out" else 1.0 / shape[0]) + 0.3 * normal
         elif name.endswith("f.b"):
             values = 2.5 + normal
         elif last == "lower":
@@ -165,7 +164,7 @@ def random_weights(config: dict, seed: int, sharp: bool = False) -> dict[str, to
         elif last == "act":
             values = np.array([0.8, -0.5, 0.6, 0.1]) + 0.2 * normal
         elif last == "canon1" or last == "conv":
-            values = 0.5 * normal
+            values = 0.4 * normal
         elif last == "b":
             values = 0.3 * normal
         elif last == "embed":
@@ -173,18 +172,18 @@ def random_weights(config: dict, seed: int, sharp: bool = False) -> dict[str, to
         elif last == "router":
             values = 3.0 * normal / np.sqrt(shape[1])
         elif last in ("q", "k") and ".mix." in name:
-            values = (5.0 if sharp else 1.7) * normal / np.sqrt(shape[1])
+            values = 1.3 * normal / np.sqrt(shape[1])
         else:
             values = normal / np.sqrt(shape[-1])
         tensors[name] = torch.from_numpy(np.asarray(values)).to(torch.bfloat16)
     return tensors
 
 
-def write_model(directory: Path, config: dict, seed: int, sharp: bool = False) -> tuple[Path, dict[str, torch.Tensor]]:
+def write_model(directory: Path, config: dict, seed: int) -> tuple[Path, dict[str, torch.Tensor]]:
     """Writes the folder; returns it and the weights in float64 (the bfloat16 values) for the plain implementation."""
     directory = Path(directory)
     directory.mkdir(parents=True, exist_ok=True)
-    tensors = random_weights(config, seed, sharp)
+    tensors = random_weights(config, seed)
     (directory / "config.json").write_text(json.dumps(config, indent=1))
     write_safetensors(directory / "model.safetensors", tensors)
     return directory, {name: tensor.to(torch.float64) for name, tensor in tensors.items()}
