@@ -316,10 +316,12 @@ def plan_flops(plan, tokens: int, wanted_rows: int = 1) -> float:
             return sum(mixer_flops(branch) for _, branch, _ in spec.branches)
         if isinstance(spec, AttentionSpec):
             value_dim = spec.value_dim or spec.head_dim
-            rows = (spec.num_heads + spec.num_groups) * spec.head_dim + spec.num_groups * value_dim + spec.num_heads * value_dim
+            maps = 2 if spec.differential is not None else 1   # two maps over the same values
+            groups = 0 if spec.borrows_kv else spec.num_groups
+            rows = (spec.num_heads + groups) * maps * spec.head_dim + groups * value_dim + spec.num_heads * value_dim
             window = spec.window or tokens
             pairs = sum(min(position + 1, window + spec.keep_first) for position in range(tokens))
-            return 2.0 * rows * spec.model_dim * tokens + 2.0 * spec.num_heads * (spec.head_dim + value_dim) * pairs
+            return 2.0 * rows * spec.model_dim * tokens + 2.0 * spec.num_heads * maps * (spec.head_dim + value_dim) * pairs
         if isinstance(spec, LatentAttentionSpec):
             # projections, the queries taken into the latent's space and the sums taken out of it, scores and sums over latent + rope channels
             heads, full = spec.num_heads, spec.latent_dim + spec.rope_dim
@@ -336,7 +338,7 @@ def plan_flops(plan, tokens: int, wanted_rows: int = 1) -> float:
             return per_token * tokens
         if isinstance(spec, LinearAttentionSpec):
             # q, k, v, gate and out projections, the decay's bottleneck, and two passes over a head's state per token
-            rows = 2 * spec.num_heads * spec.key_dim + 3 * spec.num_heads * spec.value_dim + spec.decay_rank
+            rows = 2 * spec.num_heads * spec.key_dim + (2 if spec.gate_activation == "none" else 3) * spec.num_heads * spec.value_dim + spec.decay_rank
             per_token = 2.0 * rows * spec.model_dim + 2.0 * spec.num_heads * spec.key_dim * spec.decay_rank + 4.0 * spec.num_heads * spec.key_dim * spec.value_dim
             return per_token * tokens
         if isinstance(spec, PooledWindowAttentionSpec):
@@ -374,7 +376,9 @@ def run_compare(arguments, peaks: dict, peak_source: str, families: tuple[str, .
     `--config vivulorn-compare`: the Vivulorn shapes beside the Tudulix shapes (attention, latent attention, a repeated stretch)
     and the Vuvulorn shapes (the delta rule, dense feed-forwards).
     `--config zozenex-compare`: the Zozenex shapes beside the Vuvulorn shapes (attention under a window beside a recurrence with a
-    matrix state, routed experts) and the Tudulix shapes (every layer routed, a shared expert)."""
+    matrix state, routed experts) and the Tudulix shapes (every layer routed, a shared expert).
+    `--config mozetar-compare`: the Mozetar shapes beside the Zozenex shapes (linear attention, routed experts) and the Vivulorn shapes
+    (attention over all positions, dense feed-forwards without a gate)."""
     import torch
 
     from lalamo_b200.config import config_from_dict
@@ -555,8 +559,8 @@ def main() -> int:
     parser.add_argument("--steps", type=int, default=500)
     parser.add_argument("--warmup", type=int, default=10)
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    parser.add_argument("--compare-sizes", default="350m,1.2b", help="the sizes --config vuvulorn-compare, tudulix-compare, vivulorn-compare and zozenex-compare measure")
-    parser.add_argument("--config", default="lfm2-1.2b-decode", choices=["lfm2-1.2b-decode", "lfm2-350m-mixed", "lfm2-700m-long", "vuvulorn-compare", "tudulix-compare", "vivulorn-compare", "zozenex-compare"],
+    parser.add_argument("--compare-sizes", default="350m,1.2b", help="the sizes --config vuvulorn-compare, tudulix-compare, vivulorn-compare, zozenex-compare and mozetar-compare measure")
+    parser.add_argument("--config", default="lfm2-1.2b-decode", choices=["lfm2-1.2b-decode", "lfm2-350m-mixed", "lfm2-700m-long", "vuvulorn-compare", "tudulix-compare", "vivulorn-compare", "zozenex-compare", "mozetar-compare"],
                         help="lfm2-1.2b-decode (default): the decode step and its points; lfm2-350m-mixed: 64 requests with prompts of 128 to 2,048 "
                              "tokens and 256 new tokens through the scheduler; lfm2-700m-long: 16,384-token prompts at batch 1 and 8, then 512 decode steps")
     parser.add_argument("--batch", type=int, default=8)
@@ -601,6 +605,8 @@ def main() -> int:
         return run_compare(arguments, peaks, peak_source, families=("vivulorn", "tudulix", "vuvulorn"))
     if arguments.config == "zozenex-compare":
         return run_compare(arguments, peaks, peak_source, families=("zozenex", "vuvulorn", "tudulix"))
+    if arguments.config == "mozetar-compare":
+        return run_compare(arguments, peaks, peak_source, families=("mozetar", "zozenex", "vivulorn"))
     if arguments.requests:
         requests, prompt_length, new_tokens = (int(part) for part in arguments.requests.split(","))
         engine, config = build_engine(max_tokens=requests * (prompt_length + new_tokens + 64), max_requests=max(requests, 2), max_batch_tokens=2048)

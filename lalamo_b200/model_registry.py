@@ -191,6 +191,27 @@ def _zozenex_shape(width: int, layers: int, heads: int, kv_heads: int, linear_he
     }
 
 
+def _mozetar_shape(width: int, layers: int, heads: int, kv_heads: int, linear_heads: int, linear_dim: int, linear_vdim: int, ff: int, experts: int, top: int) -> dict[str, Any]:
+    """A Mozetar shape for the random-weights mode: four residual streams, convolutions of four taps; layers in the order differential attention
+    (half as many heads as the window attention has, two maps of 64 channels each over values of 128), window attention with heads of 64
+    under 1,024 tokens, HGRN2, window attention on the keys and values of the one before it; dense feed-forwards of ``ff`` columns (two
+    matrices) in turn with routed ones of as many weights a token (``top`` experts of three matrices)."""
+    differential = {"heads": heads // 2, "kv_heads": kv_heads // 2, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4, "q_temp": {"coef": 0.1, "every": 4096}}
+    window = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125, "conv": 4, "mask": {"size": 1024},
+              "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    hgrn2 = {"heads": linear_heads, "dim": linear_dim, "vdim": linear_vdim}
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": ff * 2 // 3 // top}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+
+    def entry(index: int) -> dict[str, Any]:
+        kind = index % 4
+        mixer = (differential, window, hgrn2, {**window, "kv_from": index - 2})[kind]
+        return {"type": ("attention", "attention_2", "hgrn2", "attention_2")[kind], "mixer": mixer, "mlp": routed if index % 2 else dense}
+
+    return {"architecture": "Mozetar", "vocab": 65536, "width": width, "streams": 4, "canon": {"taps": 4}, "norm": {"eps": 1e-5},
+            "layers": [entry(index) for index in range(layers)]}
+
+
 # Shapes of the published checkpoints, and Vuvulorn shapes of the same widths and depths, for the random-weights mode
 # (no weights are downloaded).
 PRESETS: dict[str, dict[str, Any]] = {
@@ -208,4 +229,7 @@ PRESETS: dict[str, dict[str, Any]] = {
     # 16 layers; 3 routed experts + the shared one hold in their two matrices each what the three of a gated feed-forward of 4,608 (8,192) columns hold
     "zozenex-350m": _zozenex_shape(1024, 16, 16, 4, 8, 64, 128, 1728, 16, 3),
     "zozenex-1.2b": _zozenex_shape(2048, 16, 16, 4, 8, 128, 128, 3072, 16, 3),
+    # 16 layers; a dense feed-forward's two matrices (and the three of each of a token's four experts together) hold what the three of a gated one of 4,608 (8,192) columns hold
+    "mozetar-350m": _mozetar_shape(1024, 16, 16, 4, 8, 64, 128, 6912, 16, 4),
+    "mozetar-1.2b": _mozetar_shape(2048, 16, 16, 4, 8, 128, 128, 12288, 16, 4),
 }
