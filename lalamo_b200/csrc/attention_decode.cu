@@ -12,11 +12,11 @@
 //   * keys: column n of 8-key block b stands for key 4*(n/2) + 2*b + n%2 of the 16, so that lane t
 //     holds probabilities of keys 4t..4t+3, which are contiguous in the transposed value page.
 // Keys are [page][row][group][hd]; values are transposed, [page][group][hd][row]; page_size % 16 == 0.
-// Kernels with GENERAL = false take key and value heads of HD channels each; with GENERAL = true key heads of up to HD channels (a
-// multiple of 16), value heads of up to HD (a multiple of 8), several key heads over one value head, float32 output, and rows of the
+// KIND 0 takes key and value heads of HD channels each.  KIND 1 and 2 take several key heads over one value head, float32 output, and rows of the
 // cache that hold the keys of two attention maps side by side: a group's query heads are then those of the first map, which
 // meet the row's first half, and those of the second, which meet its second half (their other half counts as zeros), so that
-// both maps read keys and values once.
+// both maps read keys and values once; KIND 1 cache rows' keys of up to HD channels (a multiple of 16) and value heads of up to HD (a multiple of 8),
+// KIND 2 both of just HD.
 // Partial results (max, sum, unnormalised output per split) go to scratch; a second kernel merges
 // them in split order, so the result does not depend on the batch or on the grid.
 #include "common.cuh"
@@ -66,7 +66,7 @@ struct DecodeParams {
     // >= 0: the kernel is launched to start before the kernel before it has finished, and the newest `fresh_keys`
     // positions a token sees may still be written by that kernel; it reads the older ones while it waits.
     int fresh_keys;
-    // GENERAL only (else key_dim = value_dim = HD, keys_per_value 1, the rest 0)
+    // KIND 1 and 2 only (else key_dim = value_dim = HD, keys_per_value 1, the rest 0)
     int key_dim, value_dim;   // channels of a cache row's keys (both maps' together with two_maps) and of a value head
     int keys_per_value;       // key heads that share a value head
     int two_maps, out_float;
@@ -92,11 +92,11 @@ struct DecodeLaneSources {
     int value_step;                 // elements from a lane's value row to its next (8 channels on)
 };
 
-template <int HD, bool GENERAL>
+template <int HD, int KIND>
 __device__ __forceinline__ DecodeLaneSources decode_lane_sources(const DecodeParams& p, int group, int lane) {
     const int g = lane >> 2, t = lane & 3;
-    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
-    const int value_groups = GENERAL ? p.num_groups / p.keys_per_value : p.num_groups, value_group = GENERAL ? group / p.keys_per_value : group;
+    const int kd = KIND == 1 ? p.key_dim : HD, vd = KIND == 1 ? p.value_dim : HD;
+    const int value_groups = KIND ? p.num_groups / p.keys_per_value : p.num_groups, value_group = KIND ? group / p.keys_per_value : group;
     DecodeLaneSources sources;
     sources.key_row_stride = p.num_groups * kd;
     sources.key_page_stride = static_cast<size_t>(p.page_size) * sources.key_row_stride;
@@ -135,7 +135,7 @@ __device__ __forceinline__ void async_copy_8(void* shared_destination, const voi
 }
 
 // Starts the copies of a 16-key block (rows `in_page`.. of `page`; page -1: zeros) into `stage`.
-template <int HD, bool GENERAL>
+template <int HD, int KIND>
 __device__ __forceinline__ void issue_fragments(unsigned char* stage, const DecodeLaneSources& sources, int page, int in_page, int lane, int kd, int vd, bool& bad) {
     unsigned char* keys = stage;
     unsigned char* values = stage + HD * 32;
@@ -150,7 +150,7 @@ __device__ __forceinline__ void issue_fragments(unsigned char* stage, const Deco
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
         const __nv_bfloat16* row = sources.keys[b] + key_offset;
-        if constexpr (GENERAL) {
+        if constexpr (KIND == 1) {
 #pragma unroll
             for (int j = 0; j < HD / 16; ++j) {
                 if (16 * j < kd) async_copy_8(keys + ((b * (HD / 16) + j) * 32 + lane) * 8, reinterpret_cast<const uint2*>(row) + j);
@@ -166,18 +166,18 @@ __device__ __forceinline__ void issue_fragments(unsigned char* stage, const Deco
     const __nv_bfloat16* source = sources.values + page * sources.value_page_stride + in_page;
 #pragma unroll
     for (int n = 0; n < HD / 8; ++n) {
-        if (GENERAL && 8 * n >= vd) break;
+        if (KIND == 1 && 8 * n >= vd) break;
         async_copy_8(values + (n * 32 + lane) * 8, source);
         source += sources.value_step;
     }
 }
 
 // Reads this lane's key fragments of a stage whose copies have arrived: k[8-key block][channel block][b0, b1].
-template <int HD, bool GENERAL>
+template <int HD, int KIND>
 __device__ __forceinline__ void read_key_fragments(uint32_t (&k)[2][HD / 16][2], const unsigned char* stage, int lane) {
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
-        if constexpr (HD % 32 == 0 && !GENERAL) {
+        if constexpr (HD % 32 == 0 && KIND != 1) {
 #pragma unroll
             for (int j = 0; j < HD / 32; ++j) {
                 const uint4 loaded = *reinterpret_cast<const uint4*>(stage + ((b * (HD / 32) + j) * 32 + lane) * 16);
@@ -210,7 +210,7 @@ __device__ __forceinline__ void read_value_fragments(uint32_t (&v)[HD / 8][2], c
 }
 
 // grid (splits, groups * row_tiles, tokens), kDecodeWarps warps.
-template <int HD, bool GENERAL>
+template <int HD, int KIND>
 __global__ void __launch_bounds__(kDecodeWarps * 32, HD <= 64 ? 4 : 1)   // head size 64: 128 registers, four CTAs per SM
 attention_decode_kernel(const DecodeParams p) {
     const int split = blockIdx.x, place = blockIdx.z;
@@ -236,7 +236,7 @@ attention_decode_kernel(const DecodeParams p) {
     const int end = min(begin + p.blocks_per_split, kept_blocks + last_block - first_block + 1);
     const int rows_here = min(16, heads_per_group - row_tile * 16);
     const int head_base = group * heads_per_group + row_tile * 16;
-    const int kd = GENERAL ? p.key_dim : HD, vd = GENERAL ? p.value_dim : HD;
+    const int kd = KIND == 1 ? p.key_dim : HD, vd = KIND == 1 ? p.value_dim : HD;
 
     uint32_t q_frag[HD / 16][4];
     float out[HD / 8][4];
@@ -251,7 +251,7 @@ attention_decode_kernel(const DecodeParams p) {
     extern __shared__ __align__(16) unsigned char ring_memory[];
     unsigned char* ring = ring_memory + warp * Ring::kWarpBytes;
     const int count = end > begin + warp ? (end - begin - warp + kDecodeWarps - 1) / kDecodeWarps : 0;   // this warp's blocks: begin + warp + 4 i
-    const DecodeLaneSources sources = decode_lane_sources<HD, GENERAL>(p, group, lane);
+    const DecodeLaneSources sources = decode_lane_sources<HD, KIND>(p, group, lane);
     int table_first = 0;
     int lane_in_page = 0;
     int lane_page = lane < count ? decode_page_of(p, segment, block_of(begin + warp + kDecodeWarps * lane), lane_in_page) : -1;
@@ -263,7 +263,7 @@ attention_decode_kernel(const DecodeParams p) {
                 table_first = issued;
                 lane_page = issued + lane < count ? decode_page_of(p, segment, block_of(begin + warp + kDecodeWarps * (issued + lane)), lane_in_page) : -1;
             }
-            issue_fragments<HD, GENERAL>(ring + issue_stage * Ring::kStageBytes, sources, __shfl_sync(0xffffffffu, lane_page, issued - table_first),
+            issue_fragments<HD, KIND>(ring + issue_stage * Ring::kStageBytes, sources, __shfl_sync(0xffffffffu, lane_page, issued - table_first),
                                 __shfl_sync(0xffffffffu, lane_in_page, issued - table_first), lane, kd, vd, bad);
             ++issued;
             issue_stage = issue_stage + 1 == Ring::kStages ? 0 : issue_stage + 1;
@@ -288,7 +288,7 @@ attention_decode_kernel(const DecodeParams p) {
         for (int half = 0; half < 2; ++half) {
             const int row = g + 8 * half;
             uint2 loaded = make_uint2(0u, 0u);
-            if constexpr (GENERAL) {
+            if constexpr (KIND != 0) {
                 // with two maps a query head has half as many channels as the cache row, and meets its map's half of it
                 const int map = p.two_maps ? 2 * (row_tile * 16 + row) / heads_per_group : 0, q_dim = p.two_maps ? kd / 2 : kd;
                 if (row < rows_here && 16 * j < kd && (!p.two_maps || map == t >> 1)) {
@@ -323,12 +323,12 @@ attention_decode_kernel(const DecodeParams p) {
             for (int b = 0; b < 2; ++b) s[which][b][0] = s[which][b][1] = s[which][b][2] = s[which][b][3] = which == 1 && !two ? -INFINITY : 0.0f;
             if (which == 0 || two) {
                 uint32_t k[2][HD / 16][2];
-                read_key_fragments<HD, GENERAL>(k, stages[which], lane);
+                read_key_fragments<HD, KIND>(k, stages[which], lane);
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
 #pragma unroll
                     for (int j = 0; j < HD / 16; ++j) {
-                        if (!GENERAL || 16 * j < kd) mma_16816(s[which][b], q_frag[j], k[b][j][0], k[b][j][1]);
+                        if (KIND != 1 || 16 * j < kd) mma_16816(s[which][b], q_frag[j], k[b][j][0], k[b][j][1]);
                     }
                 }
             }
@@ -421,7 +421,7 @@ attention_decode_kernel(const DecodeParams p) {
                 }
 #pragma unroll
                 for (int n = 0; n < HD / 8; ++n) {
-                    if (!GENERAL || 8 * n < vd) mma_16816(out[n], p_frag[which], v[n][0], v[n][1]);
+                    if (KIND != 1 || 8 * n < vd) mma_16816(out[n], p_frag[which], v[n][0], v[n][1]);
                 }
             }
         }
@@ -470,7 +470,7 @@ attention_decode_kernel(const DecodeParams p) {
             // all of the token's keys were this CTA's: what the merge kernel would make of the one partial
             const size_t place_out = (static_cast<size_t>(token) * p.num_heads + head_base + row) * vd + d;
             const float result = sum > 0.0f ? value / sum : 0.0f;
-            if (GENERAL && p.out_float) static_cast<float*>(p.out)[place_out] = result;
+            if (KIND && p.out_float) static_cast<float*>(p.out)[place_out] = result;
             else static_cast<__nv_bfloat16*>(p.out)[place_out] = __float2bfloat16_rn(result);
             continue;
         }
@@ -524,12 +524,12 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ partial_
     }
 }
 
-template <int HD, bool GENERAL>
+template <int HD, int KIND>
 int launch_decode(const DecodeParams& p, int tokens, cudaStream_t stream) {
     const int heads_per_group = p.num_heads / p.num_groups;
     const int row_tiles = (heads_per_group + 15) / 16;
     const dim3 grid(p.splits, p.num_groups * row_tiles, tokens);
-    auto kernel = attention_decode_kernel<HD, GENERAL>;
+    auto kernel = attention_decode_kernel<HD, KIND>;
     static OncePerDevice configured;
     if (allow_shared_memory(configured, kernel, DecodeRing<HD>::kBytes) != cudaSuccess) return static_cast<int>(cudaGetLastError());
     if (p.fresh_keys >= 0) {
@@ -540,10 +540,10 @@ int launch_decode(const DecodeParams& p, int tokens, cudaStream_t stream) {
     }
     if (p.splits > 1) {
         const dim3 merge_grid(p.num_heads, tokens);
-        if (GENERAL && p.out_float)
+        if (KIND && p.out_float)
             attention_decode_merge_kernel<0, float><<<merge_grid, 64, 0, stream>>>(p.partial_out, p.partial_stats, static_cast<float*>(p.out), p.token_list, p.num_heads,
                                                                                  p.splits, p.value_dim);
-        else if (GENERAL)
+        else if (KIND)
             attention_decode_merge_kernel<0, __nv_bfloat16><<<merge_grid, 64, 0, stream>>>(p.partial_out, p.partial_stats, static_cast<__nv_bfloat16*>(p.out),
                                                                                          p.token_list, p.num_heads, p.splits, p.value_dim);
         else
@@ -565,8 +565,8 @@ int lb_attention_decode_ctas_per_sm(int head_dim) {
 #define LB_DECODE_OCCUPANCY(HD)                                                                                          \
     case HD: {                                                                                                           \
         static lb::OncePerDevice configured;                                                                             \
-        if (lb::allow_shared_memory(configured, lb::attention_decode_kernel<HD, false>, lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0; \
-        if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&ctas, lb::attention_decode_kernel<HD, false>, lb::kDecodeWarps * 32,  \
+        if (lb::allow_shared_memory(configured, lb::attention_decode_kernel<HD, 0>, lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0; \
+        if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&ctas, lb::attention_decode_kernel<HD, 0>, lb::kDecodeWarps * 32,  \
                                                           lb::DecodeRing<HD>::kBytes) != cudaSuccess) return 0;          \
         return ctas;                                                                                                     \
     }
@@ -586,7 +586,7 @@ long long lb_attention_decode_scratch_floats(int tokens, int num_heads, int head
 
 // Returns 0, a CUDA error code, -1 for an unsupported type, or -2 for sizes the kernel does not take
 // (head_dim must be a multiple of 16 up to 128, page_size a multiple of 16, the scale positive).  value_dim (0: head_dim), value_groups
-// (0: num_groups), two_maps and out_float: see GENERAL above; with two_maps head_dim counts both maps' channels, num_groups the
+// (0: num_groups), two_maps and out_float: see KIND above; with two_maps head_dim counts both maps' channels, num_groups the
 // cache rows' groups and num_heads both maps' query heads; value_dim must be a multiple of 8 up to 128.
 int lb_attention_decode(const void* q, const void* k_pages, const void* v_pages, void* out, float* scratch,
                         const int* positions, const int* token_segment, const int* block_table, const int* token_list,
@@ -632,21 +632,23 @@ int lb_attention_decode(const void* q, const void* k_pages, const void* v_pages,
     p.status = status;
     p.fresh_keys = fresh_keys;
     if (general) {
+        if (head_dim == value_dim && head_dim == 64) return lb::launch_decode<64, 2>(p, tokens, stream);
+        if (head_dim == value_dim && head_dim == 128) return lb::launch_decode<128, 2>(p, tokens, stream);
         const int widest = head_dim > value_dim ? head_dim : value_dim;
-        if (widest <= 32) return lb::launch_decode<32, true>(p, tokens, stream);
-        if (widest <= 64) return lb::launch_decode<64, true>(p, tokens, stream);
-        if (widest <= 96) return lb::launch_decode<96, true>(p, tokens, stream);
-        return lb::launch_decode<128, true>(p, tokens, stream);
+        if (widest <= 32) return lb::launch_decode<32, 1>(p, tokens, stream);
+        if (widest <= 64) return lb::launch_decode<64, 1>(p, tokens, stream);
+        if (widest <= 96) return lb::launch_decode<96, 1>(p, tokens, stream);
+        return lb::launch_decode<128, 1>(p, tokens, stream);
     }
     switch (head_dim) {
-        case 16: return lb::launch_decode<16, false>(p, tokens, stream);
-        case 32: return lb::launch_decode<32, false>(p, tokens, stream);
-        case 48: return lb::launch_decode<48, false>(p, tokens, stream);
-        case 64: return lb::launch_decode<64, false>(p, tokens, stream);
-        case 80: return lb::launch_decode<80, false>(p, tokens, stream);
-        case 96: return lb::launch_decode<96, false>(p, tokens, stream);
-        case 112: return lb::launch_decode<112, false>(p, tokens, stream);
-        case 128: return lb::launch_decode<128, false>(p, tokens, stream);
+        case 16: return lb::launch_decode<16, 0>(p, tokens, stream);
+        case 32: return lb::launch_decode<32, 0>(p, tokens, stream);
+        case 48: return lb::launch_decode<48, 0>(p, tokens, stream);
+        case 64: return lb::launch_decode<64, 0>(p, tokens, stream);
+        case 80: return lb::launch_decode<80, 0>(p, tokens, stream);
+        case 96: return lb::launch_decode<96, 0>(p, tokens, stream);
+        case 112: return lb::launch_decode<112, 0>(p, tokens, stream);
+        case 128: return lb::launch_decode<128, 0>(p, tokens, stream);
         default: return -2;
     }
 }

@@ -158,7 +158,6 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(barriers + 9);
     __shared__ int failed;
 
-    allow_next_kernel();   // the out-projection that follows may ask for its weights meanwhile
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int heads_per_group = p.num_heads / p.num_groups;
     const int group = blockIdx.y, value_group = group / p.keys_per_value;
@@ -222,6 +221,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    // The out-projection that follows may ask for its weights meanwhile: it takes tensor memory of its own, so only now that this
+    // CTA has its share.
+    allow_next_kernel();
     const uint32_t tmem_base = *tmem_slot;
     const uint32_t tmem_scores = tmem_base, tmem_output = tmem_base + kTaKeys;
 

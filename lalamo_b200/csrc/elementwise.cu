@@ -456,7 +456,7 @@ __global__ void branch_norms_accumulate_kernel(float* __restrict__ residual, con
 // (powers element by element), 32-bit inside, rounded once.  The row is read twice, the second time from the caches.
 template <typename T>
 __global__ void poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ coefficients, T* __restrict__ out, int dim, float eps) {
-    __shared__ float scratch[3][33];
+    __shared__ float scratch[3][32];
     wait_for_previous_kernel();
     allow_next_kernel();
     const T* row = z + static_cast<size_t>(blockIdx.x) * dim;
@@ -485,7 +485,17 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, const float* __restric
     }
     float factor[3];
 #pragma unroll
-    for (int i = 0; i < 3; ++i) factor[i] = coefficients[i] * rsqrtf(block_sum(sums[i], scratch[i]) / static_cast<float>(dim) + eps);
+    for (int i = 0; i < 3; ++i) {   // the three sums over the block in one exchange, warps in order
+        const float sum = warp_sum(sums[i]);
+        if ((threadIdx.x & 31) == 0) scratch[i][threadIdx.x >> 5] = sum;
+    }
+    __syncthreads();
+    const int warps = (blockDim.x + 31) >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+    for (int i = 0; i < 3; ++i) {
+        const float sum = warp_sum(lane < warps ? scratch[i][lane] : 0.0f);
+        factor[i] = coefficients[i] * rsqrtf(sum / static_cast<float>(dim) + eps);
+    }
     const float constant = coefficients[3];
     auto value = [&](float v) { return fmaf(fmaf(fmaf(factor[2], v, factor[1]), v, factor[0]), v, constant); };
     if (wide) {

@@ -141,8 +141,9 @@ __device__ __forceinline__ void load_output(const StreamStep<T>& p, size_t row, 
 // One block per output row.
 constexpr int stream_step_threads(int streams) { return streams <= 4 ? 512 : 256; }   // the coefficients take registers
 
-template <typename T, int S, int V>
-__global__ void __launch_bounds__(stream_step_threads(S)) stream_step_kernel(const StreamStep<T> p) {
+// MANY: launches of many rows in blocks of at most 256 threads, of which as many as registers allow share an SM.
+template <typename T, int S, int V, bool MANY>
+__global__ void __launch_bounds__(MANY ? 256 : stream_step_threads(S), MANY ? (S <= 4 ? 4 : 1) : 1) stream_step_kernel(const StreamStep<T> p) {
     extern __shared__ __align__(16) float shared[];
     // Launched to start early; the product after it may then ask for its weights, but not before the kernel before is done.
     wait_for_previous_kernel();
@@ -246,7 +247,7 @@ int launch_stream_step(const StreamStep<T>& p, int streams, int out_rows, cudaSt
     switch (streams) {
 #define LB_STREAM_CASE(S)                                                                                                                     \
     case S: {                                                                                                                                 \
-        auto kernel = stream_step_kernel<T, S, V>;                                                                                            \
+        auto kernel = out_rows <= 64 ? stream_step_kernel<T, S, V, false> : stream_step_kernel<T, S, V, true>;                                \
         if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));          \
         error = launch_overlapped(kernel, dim3(out_rows), dim3(threads), shared, stream, p);                                                  \
         break;                                                                                                                                \
@@ -260,7 +261,11 @@ int launch_stream_step(const StreamStep<T>& p, int streams, int out_rows, cudaSt
 }
 
 // ------------------------------------------------------------------------------------------- causal convolution
-constexpr int kConvRows = 16;   // tokens per block; taps - 1 may not exceed it
+// Tokens per block; taps - 1 may not exceed them.  Few, where the number of taps is known: all of a thread's loads leave before the first sum.
+template <int TAPS>
+struct ConvRows {
+    static constexpr int kRows = TAPS > 0 ? 4 : 16;
+};
 
 // V consecutive elements, 16 bytes at a time where V elements make that much.
 template <typename T, int V>
@@ -290,9 +295,9 @@ __device__ __forceinline__ void store_pack(T* destination, const float (&v)[V]) 
     }
 }
 
-// grid (tiles of kConvRows tokens of the longest portion, portions, pieces of the channels); a thread per V channels.
+// grid (tiles of ConvRows tokens of the longest portion, portions, pieces of the channels); a thread per V channels.
 //   out_t = [x_t +] sum_j w[:, j] x_(t - taps + 1 + j), what lies before the portion from the request's state
-// A portion's first tile reads all of the state that anyone reads (taps - 1 <= kConvRows) and then moves it on: row i becomes the
+// A portion's first tile reads all of the state that anyone reads (taps - 1 <= ConvRows) and then moves it on: row i becomes the
 // portion's input at len - (taps - 1) + i, or an old row where the portion is shorter than that.  TAPS 0: any number of taps.
 template <typename T, int TAPS, int V>
 __global__ void causal_conv_kernel(const T* __restrict__ x, int x_stride, T* __restrict__ state, const float* __restrict__ weight, T* __restrict__ out,
@@ -302,7 +307,9 @@ __global__ void causal_conv_kernel(const T* __restrict__ x, int x_stride, T* __r
     allow_next_kernel();
     const int taps = TAPS > 0 ? TAPS : any_taps;
     const int segment = blockIdx.y;
-    const int first = blockIdx.x * kConvRows, length = segment_length[segment];
+    constexpr int kRows = ConvRows<TAPS>::kRows;
+    static_assert(TAPS - 1 <= kRows, "a portion's first tile reads all of the state that is read");
+    const int first = blockIdx.x * kRows, length = segment_length[segment];
     const int channel = (blockIdx.z * blockDim.x + threadIdx.x) * V;
     if (first >= length || channel >= channels) return;
     const int slot = segment_slot[segment];
@@ -311,7 +318,7 @@ __global__ void causal_conv_kernel(const T* __restrict__ x, int x_stride, T* __r
     T* own_state = good && taps > 1 ? state + static_cast<size_t>(slot) * (taps - 1) * channels + channel : nullptr;
     const T* source = x + static_cast<size_t>(segment_start[segment]) * x_stride + channel;
     T* destination = out + static_cast<size_t>(segment_start[segment]) * out_stride + channel;
-    const int end = min(length, first + kConvRows);
+    const int end = min(length, first + kRows);
     // the input at local index t, which may lie in the state
     auto input = [&](int t, float (&v)[V]) {
         if (t >= 0) {
@@ -324,31 +331,41 @@ __global__ void causal_conv_kernel(const T* __restrict__ x, int x_stride, T* __r
         }
     };
     if constexpr (TAPS > 0) {
-        float w[TAPS][V], held[TAPS][V];   // held: the last TAPS inputs, oldest first
+        float held[kRows + TAPS - 1][V];   // the inputs at first - (TAPS - 1) ... first + kRows - 1
 #pragma unroll
-        for (int i = 0; i < V; ++i) {
+        for (int r = 0; r < kRows + TAPS - 1; ++r) {
+            if (first - (TAPS - 1) + r < end) {
+                input(first - (TAPS - 1) + r, held[r]);
+            } else {
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) w[j][i] = weight[static_cast<size_t>(channel + i) * TAPS + j];
+                for (int i = 0; i < V; ++i) held[r][i] = 0.0f;
+            }
+        }
+        float w[V * TAPS];   // of this thread's channels, one after the other in memory
+        const float* own_weight = weight + static_cast<size_t>(channel) * TAPS;
+        if constexpr ((V * TAPS) % 4 == 0) {
+#pragma unroll
+            for (int i = 0; i < V * TAPS; i += 4) {
+                const float4 four = *reinterpret_cast<const float4*>(own_weight + i);
+                w[i] = four.x, w[i + 1] = four.y, w[i + 2] = four.z, w[i + 3] = four.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < V * TAPS; ++i) w[i] = own_weight[i];
         }
 #pragma unroll
-        for (int j = 0; j + 1 < TAPS; ++j) input(first - (TAPS - 1) + j, held[j + 1]);
-#pragma unroll 4
-        for (int t = first; t < end; ++t) {
+        for (int r = 0; r < kRows; ++r) {
+            if (first + r < end) {
+                float sum[V];
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) {
+                for (int i = 0; i < V; ++i) {
+                    sum[i] = 0.0f;
 #pragma unroll
-                for (int i = 0; i < V; ++i) held[j][i] = held[j + 1][i];
+                    for (int j = 0; j < TAPS; ++j) sum[i] += w[i * TAPS + j] * held[r + j][i];
+                    if (add_input) sum[i] += held[r + TAPS - 1][i];
+                }
+                store_pack<T, V>(destination + static_cast<size_t>(first + r) * out_stride, sum);
             }
-            input(t, held[TAPS - 1]);
-            float sum[V];
-#pragma unroll
-            for (int i = 0; i < V; ++i) {
-                sum[i] = 0.0f;
-#pragma unroll
-                for (int j = 0; j < TAPS; ++j) sum[i] += w[j][i] * held[j][i];
-                if (add_input) sum[i] += held[TAPS - 1][i];
-            }
-            store_pack<T, V>(destination + static_cast<size_t>(t) * out_stride, sum);
         }
     } else {
         for (int t = first; t < end; ++t) {
@@ -382,11 +399,12 @@ int launch_causal_conv(const void* x, int x_stride, void* state, const float* we
                        cudaStream_t stream) {
     const int threads_needed = (channels + V - 1) / V;
     const int threads = threads_needed >= 128 ? 128 : (threads_needed + 31) / 32 * 32;
-    const dim3 grid((max_length + kConvRows - 1) / kConvRows, segments, (threads_needed + threads - 1) / threads);
     auto kernel = causal_conv_kernel<T, 0, V>;
     if (taps == 2) kernel = causal_conv_kernel<T, 2, V>;
     if (taps == 3) kernel = causal_conv_kernel<T, 3, V>;
     if (taps == 4) kernel = causal_conv_kernel<T, 4, V>;
+    const int rows = taps >= 2 && taps <= 4 ? ConvRows<4>::kRows : ConvRows<0>::kRows;
+    const dim3 grid((max_length + rows - 1) / rows, segments, (threads_needed + threads - 1) / threads);
     const cudaError_t error = launch_overlapped(kernel, grid, dim3(threads), 0, stream, static_cast<const T*>(x), x_stride, static_cast<T*>(state), weight,
                                                 static_cast<T*>(out), out_stride, channels, taps, add_input, segment_start, segment_length, segment_slot, num_slots,
                                                 status);
@@ -451,7 +469,7 @@ int lb_causal_conv(const void* x, int x_stride, void* state, const float* weight
                    const int* segment_start, const int* segment_length, const int* segment_slot, int segments, int max_length, int num_slots, int dtype,
                    int* status, cudaStream_t stream) {
     if (segments == 0 || max_length == 0 || channels == 0) return 0;
-    if (taps < 1 || taps - 1 > lb::kConvRows) return -2;
+    if (taps < 1 || taps - 1 > lb::ConvRows<0>::kRows) return -2;
     const bool even8 = channels % 8 == 0 && x_stride % 8 == 0 && out_stride % 8 == 0;
     const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(state)) & 15) == 0;
     if (dtype == lb::kBFloat16) {
