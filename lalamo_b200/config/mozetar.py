@@ -11,7 +11,7 @@ three, in an order the configuration lists:
 * ``"attention_2"``: grouped attention under a sliding window, q, k and v convolved over time after their projections, rotary
   positions on neighbouring channels of part of q and k with frequencies slowed down for long contexts; with ``kv_from`` it has no
   keys and values of its own and reads the named layer's;
-* ``"hgrn2"``: linear attention whose forget gate, bounded from below per channel, also decides what is written.
+* ``"hgrn2"``: linear attention whose decay is a forget gate with a lower bound per channel, and whose keys are what that gate leaves free.
 
 The feed-forward is dense (``W_down poly(W_up h)`` with biases, ``poly`` a polynomial of normalised powers), a mixture of gated silu
 experts (softmax scores, the best groups of neighbours by their largest score, the chosen scores over their sum), or absent.

@@ -341,7 +341,7 @@ class GatedMLPSpec(FeedForwardSpec):
 @dataclass(frozen=True)
 class DenseMLPSpec(FeedForwardSpec):
     """``down(act(up(x) + b_up)) + b_down``: two projections, no gate.  ``activation``: ``"gelu"`` (the exact gelu,
-    ``0.5 z (1 + erf(z / sqrt 2))``), ``"silu"``, ``"identity"``, or ``"poly_norm"``: ``a N(z) + b N(z^2) + c N(z^3) + e`` with four learned
+    ``0.5 z (1 + erf(z / sqrt 2))``), ``"silu"``, ``"identity"``, or ``"poly_norm"``: ``c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3`` with four learned
     numbers, powers element by element and ``N(v) = v / sqrt(mean(v^2) + norm_eps)`` over a token's hidden values."""
 
     kind: ClassVar[str] = "dense_mlp"

@@ -128,7 +128,7 @@ def convolved_attention(h: torch.Tensor, w: dict, cfg: dict, shared: dict, index
 
 
 def forget_recurrence(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, state: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
-    """``S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T; o_t = S_t^T q_t`` per head; returns the read-outs and the last state."""
+    """A state ``S[i, j]`` per head becomes ``f[i] S[i, j] + (1 - f[i]) v[j]`` at every token and is read as ``sum_i q[i] S[i, j]``; returns the read-outs and the last state."""
     tokens, heads, dk = q.shape
     state = torch.zeros(heads, dk, v.shape[-1], dtype=DT) if state is None else state.clone()
     out = torch.zeros(tokens, heads, v.shape[-1], dtype=DT)
