@@ -15,12 +15,14 @@ from .plan import (
     InputConvSpec,
     LatentAttentionSpec,
     LayerNormSpec,
+    LayerScaleSpec,
     LinearAttentionSpec,
     LlamaScaling,
     MixerSpec,
     ModelPlan,
     NormSpec,
     OutputNormBlockSpec,
+    ParallelBlockSpec,
     ParallelMixerSpec,
     PooledWindowAttentionSpec,
     PositionSpec,
@@ -38,6 +40,7 @@ from .plan import (
 from .tudulix import TudulixConfig
 from .vivulorn import VivulornConfig
 from .vuvulorn import VuvulornConfig
+from .zevetar import ZevetarConfig
 from .zozenex import ZozenexConfig
 from .registry import architectures, config_from_dict, load_config, register_architecture
 
@@ -47,6 +50,7 @@ register_architecture("Tudulix", TudulixConfig)
 register_architecture("Vivulorn", VivulornConfig)
 register_architecture("Zozenex", ZozenexConfig)
 register_architecture("Mozetar", MozetarConfig)
+register_architecture("Zevetar", ZevetarConfig)
 
 __all__ = [
     "AttentionSpec",
@@ -61,6 +65,7 @@ __all__ = [
     "InputConvSpec",
     "LatentAttentionSpec",
     "LayerNormSpec",
+    "LayerScaleSpec",
     "Lfm2Config",
     "LinearAttentionSpec",
     "LlamaScaling",
@@ -69,6 +74,7 @@ __all__ = [
     "MozetarConfig",
     "NormSpec",
     "OutputNormBlockSpec",
+    "ParallelBlockSpec",
     "ParallelMixerSpec",
     "PooledWindowAttentionSpec",
     "PositionSpec",
@@ -86,6 +92,7 @@ __all__ = [
     "VivulornConfig",
     "VuvulornConfig",
     "YarnScaling",
+    "ZevetarConfig",
     "ZozenexConfig",
     "architectures",
     "config_from_dict",

@@ -30,12 +30,14 @@ __all__ = [
     "InputConvSpec",
     "LatentAttentionSpec",
     "LayerNormSpec",
+    "LayerScaleSpec",
     "LinearAttentionSpec",
     "LlamaScaling",
     "MixerSpec",
     "ModelPlan",
     "NormSpec",
     "OutputNormBlockSpec",
+    "ParallelBlockSpec",
     "ParallelMixerSpec",
     "PooledWindowAttentionSpec",
     "PositionSpec",
@@ -130,6 +132,8 @@ class RopeSpec(PositionSpec):
     pairing: str = "half"
     # stretched frequencies (and, under YarnScaling, a factor on sines and cosines)
     scaling: YarnScaling | LlamaScaling | None = None
+    # True: the frequencies are worked out in 64-bit and rounded once (False: in 32-bit, as the reference's are; scaled ones always in 64-bit)
+    exact: bool = False
 
 
 @dataclass(frozen=True)
@@ -195,7 +199,10 @@ class LatentAttentionSpec(MixerSpec):
     shared by all heads; per head the unrotated key is ``W_uk c`` (``head_dim`` channels), the value ``W_uv c``
     (``value_dim``); a query head is ``[head_dim unrotated, rope_dim rotated]``; the score is
     ``(q_plain . k_plain + q_rot . r) * scale``.  Only ``c`` and ``r`` are cached.  ``gated``: the heads' outputs are
-    multiplied by ``sigmoid(W_gate h)`` before the out-projection."""
+    multiplied by ``sigmoid(W_gate h)`` before the out-projection.  ``query_rank`` > 0: the queries go through a latent of their own,
+    ``q = W_q_up norm(W_q_down h)`` (``query_norm``, a plain weight); 0: ``q = W_q h``.  A factor that ``position`` puts on sines and
+    cosines applies to the rotated parts of both sides.  ``borrows_kv``: the mixer leaves nothing behind; it reads the rows that the
+    schedule entry named by ``cache_from`` writes, with its own queries, per-head projections, window and scale."""
 
     kind: ClassVar[str] = "latent_attention"
     model_dim: int = 0
@@ -210,6 +217,9 @@ class LatentAttentionSpec(MixerSpec):
     scale: float | None = None  # None -> (head_dim + rope_dim) ** -0.5
     gated: bool = False
     sink: bool = False  # a learned number per head whose exponential joins the softmax's denominator (no key, no value, not scaled)
+    query_rank: int = 0
+    query_norm: NormSpec | None = None
+    borrows_kv: bool = False
 
 
 @dataclass(frozen=True)
@@ -254,7 +264,8 @@ class LinearAttentionSpec(MixerSpec):
     multiplied by ``silu(W_g h)`` (or ``sigmoid``, ``gate_activation``; ``"none"``: no gate) and projected out.  ``decay="forget"``
     (HGRN2): one forget gate per head and key channel, ``a = l + (1 - l) sigmoid(W_f h + b)`` with a learned lower bound ``l``, which
     also says what is written, ``k = 1 - a`` (there is no key projection).  ``scaled="none"``: neither is scaled;
-    ``query_activation="silu"``: q is silu of its projection.  State, decays and their logarithms,
+    ``query_activation="silu"``: q is silu of its projection.  ``position`` rotates (part of) every head of q and k, before any
+    scale.  State, decays and their logarithms, positions, angles,
     the recurrence's inputs and the read-out norm are 32-bit."""
 
     kind: ClassVar[str] = "linear_attention"
@@ -271,6 +282,7 @@ class LinearAttentionSpec(MixerSpec):
     norm_eps: float = 1e-5
     gate_activation: str = "silu"
     query_activation: str = "identity"
+    position: PositionSpec | None = None
 
 
 @dataclass(frozen=True)
@@ -363,7 +375,8 @@ class RoutedMLPSpec(FeedForwardSpec):
     ``"sigmoid_limit"`` activation (see :class:`GatedMLPSpec`).  ``shared``: a dense feed-forward that every token
     runs besides, added to the experts' weighted sum (``shared_gate``: times ``sigmoid(w_sg . h)``, one number per token).
     ``gated=False``: the experts are ``down(act(up(x)))`` without a gate.  ``choice_bias``: a learned number per expert added to
-    the scores where experts (and groups) are ranked, not where they weigh.  ``weight_scale`` multiplies the weights."""
+    the scores where experts (and groups) are ranked, not where they weigh.  ``weight_scale`` multiplies the weights.
+    ``weigh_input``: a weight multiplies its expert's input, ``sum_k expert_k(w_k x)``, not its output."""
 
     kind: ClassVar[str] = "routed_mlp"
     model_dim: int = 0
@@ -384,6 +397,7 @@ class RoutedMLPSpec(FeedForwardSpec):
     weight_scale: float = 1.0
     shared_gate: bool = False
     group_score: str = "two_largest"
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
@@ -420,6 +434,14 @@ class HyperBlockSpec:
 
 
 @dataclass(frozen=True)
+class LayerScaleSpec:
+    """A learned vector of ``dim`` elements that multiplies a sublayer's output element by element (32-bit)."""
+
+    kind: ClassVar[str] = "layer_scale"
+    dim: int = 0
+
+
+@dataclass(frozen=True)
 class OutputNormBlockSpec:
     """A block whose sublayers read the residual stream itself and whose norms sit on the sublayers'
     outputs: ``x <- x + mixer_norm(mixer(x)); x <- x + ffn_norm(ffn(x))`` (``ffn=None``: no second half)."""
@@ -443,6 +465,20 @@ class SandwichBlockSpec:
     ffn: FeedForwardSpec | None = None
     ffn_out_norm: NormSpec | None = None
     arrangement: str = "sandwich_norm"
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """A block of one norm whose two sublayers read the same normed input and are added at once:
+    ``h = norm(x); y = x + mixer(h) + ffn(h)`` (``ffn=None``: the mixer alone).  ``mixer_scale`` / ``ffn_scale``: the sublayer's output
+    is multiplied element by element by a learned vector before the sum."""
+
+    norm: NormSpec
+    mixer: MixerSpec
+    ffn: FeedForwardSpec | None = None
+    mixer_scale: LayerScaleSpec | None = None
+    ffn_scale: LayerScaleSpec | None = None
+    arrangement: str = "parallel"
 
 
 @dataclass(frozen=True)
@@ -516,7 +552,7 @@ class ScheduleEntry:
 class ModelPlan:
     vocab_size: int
     model_dim: int
-    layers: tuple[BlockSpec | HyperBlockSpec | OutputNormBlockSpec | SandwichBlockSpec, ...]
+    layers: tuple[BlockSpec | HyperBlockSpec | OutputNormBlockSpec | ParallelBlockSpec | SandwichBlockSpec, ...]
     final_norm: NormSpec
     tie_embeddings: bool = True
     embedding_scale: float | None = None

@@ -5,6 +5,7 @@
 //
 //   latent_prepare           norm of the latent, rotation of the shared key part and of the queries' rotated parts,
 //                            the page write, and the queries laid out [token][head][latent | rope]
+//   latent_down              where the queries go through a latent of their own: its norm, and the page write, in one step
 //   latent_attention_plain   one block per (token, head): 32-bit scores, softmax and sums; the 32-bit path's
 //                            attention and the reference for the tensor-core kernel
 //   gate_heads               heads' values [head][token][vdim] times sigmoid(gate), laid out [token][head * vdim]
@@ -31,19 +32,87 @@ __device__ __forceinline__ T* latent_row(T* pages, const int* block_table, const
     return pages + row * (layout.latent + layout.rope);
 }
 
+// Writes the token's row, [T(norm(down[:latent]) * (w + offset)) | rope(down[latent:])], with a whole block; `cosines` and `sines` (already
+// times the factor the position encoding puts on them) are in shared memory when the first block-wide sum has passed.
+template <typename T>
+__device__ __forceinline__ void write_latent_row(const T* __restrict__ row, T* __restrict__ dst, const float* __restrict__ norm_weight, float eps, float scale_offset,
+                                                 const float* cosines, const float* sines, float* scratch, int latent, int half, int* status) {
+    float squares = 0.0f;
+    for (int d = threadIdx.x; d < latent; d += blockDim.x) {
+        const float v = to_float(row[d]);
+        squares += v * v;
+    }
+    const float total = block_sum(squares, scratch);   // also orders the writes to cosines[] and sines[]
+    if (dst == nullptr) {
+        if (threadIdx.x == 0) report_error(status, kBadPage);
+        return;
+    }
+    const float inv = rsqrtf(total / static_cast<float>(latent) + eps);
+    for (int d = threadIdx.x; d < latent; d += blockDim.x) dst[d] = from_float<T>(to_float(row[d]) * inv * (norm_weight[d] + scale_offset));
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float u = to_float(row[latent + i]), v = to_float(row[latent + half + i]);
+        dst[latent + i] = from_float<T>(u * cosines[i] - v * sines[i]);
+        dst[latent + half + i] = from_float<T>(v * cosines[i] + u * sines[i]);
+    }
+}
+
+// sines and cosines of one position's angles, times `factor`
+__device__ __forceinline__ void latent_turns(float* cosines, float* sines, const float* __restrict__ inv_freq, int position, int half, float factor) {
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf(static_cast<float>(position) * inv_freq[i], &s, &c);
+        sines[i] = s * factor;
+        cosines[i] = c * factor;
+    }
+}
+
+// grid (tokens, 1 or 2), what lies between the down-projections and the queries' up-projection.  Block (t, 0): the query latent's norm,
+// q_latent [tokens][q_latent_stride] = T(norm(q_down[:q_rank]) * w), zeros behind q_rank.  Block (t, 1), for layers that leave rows
+// behind: the token's row (see write_latent_row).  q_down and down are column slices of one product, row_stride elements a token.
+template <typename T>
+__global__ void latent_down_kernel(const T* __restrict__ q_down, const T* __restrict__ down, int row_stride, T* __restrict__ q_latent, int q_latent_stride,
+                                   int q_rank, const float* __restrict__ q_norm_weight, float q_eps, T* __restrict__ pages, const float* __restrict__ norm_weight,
+                                   float eps, float scale_offset, const float* __restrict__ inv_freq, float factor, const int* __restrict__ positions,
+                                   const int* __restrict__ token_segment, const int* __restrict__ block_table, LatentLayout layout, int* status) {
+    extern __shared__ float shared[];
+    wait_for_previous_kernel();
+    allow_next_kernel();
+    const int half = layout.rope / 2, token = blockIdx.x;
+    float* cosines = shared;
+    float* sines = shared + half;
+    float* scratch = sines + half;   // 33
+    if (blockIdx.y == 1) {
+        const int position = positions[token];
+        latent_turns(cosines, sines, inv_freq, position, half, factor);
+        write_latent_row(down + static_cast<size_t>(token) * row_stride, latent_row(pages, block_table, layout, token_segment[token], position), norm_weight, eps,
+                         scale_offset, cosines, sines, scratch, layout.latent, half, status);
+        return;
+    }
+    const T* row = q_down + static_cast<size_t>(token) * row_stride;
+    T* dst = q_latent + static_cast<size_t>(token) * q_latent_stride;
+    float squares = 0.0f;
+    for (int d = threadIdx.x; d < q_rank; d += blockDim.x) {
+        const float v = to_float(row[d]);
+        squares += v * v;
+    }
+    const float inv = rsqrtf(block_sum(squares, scratch) / static_cast<float>(q_rank) + q_eps);
+    for (int d = threadIdx.x; d < q_latent_stride; d += blockDim.x) dst[d] = from_float<T>(d < q_rank ? to_float(row[d]) * inv * q_norm_weight[d] : 0.0f);
+}
+
 // grid (tokens, head blocks + 1): blocks (t, b) lay out token t's query heads, block (t, head blocks) writes the token's row.
 //   q        [tokens][q_stride]: head h at h * (head_dim + rope), its last `rope` channels are rotated
 //   q_latent [heads][tokens][latent]: the heads' unrotated parts taken into the latent's space
 //   down     [tokens][down_stride]: [latent | rope]
 //   q_out    [tokens][heads][latent + rope]
 //   pages    [page][row][latent + rope]: row = [T(norm(down[:latent]) * (w + offset)) | rope(down[latent:])]
-// The rotation pairs channel i with i + rope / 2: (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = position * inv_freq[i].
+// The rotation pairs channel i with i + rope / 2: (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = position * inv_freq[i], sines and
+// cosines times `factor`.  grid.y without the last block where nothing writes rows (write_kv 0).
 template <typename T>
 __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ q_latent, const T* __restrict__ down, int down_stride,
                                       T* __restrict__ q_out, T* __restrict__ pages, const float* __restrict__ norm_weight, float eps, float scale_offset,
                                       const float* __restrict__ inv_freq, const int* __restrict__ positions, const int* __restrict__ token_segment,
                                       const int* __restrict__ block_table, LatentLayout layout, int tokens, int num_heads, int head_dim, int write_kv,
-                                      int* status) {
+                                      int* status, float factor) {
     extern __shared__ float shared[];
     const int half = layout.rope / 2, latent = layout.latent, rope = layout.rope;
     float* cosines = shared;            // half
@@ -51,10 +120,9 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, con
     float* scratch = sines + half;      // 33
     // blocks (t, 0 .. head_blocks - 1) take heads_per_block heads each (one where the latent parts are copied, all where only
     // the rotated parts are written), block (t, head_blocks) the token's row
-    const int token = blockIdx.x, unit = blockIdx.y, head_blocks = gridDim.y - 1, heads_per_block = (num_heads + head_blocks - 1) / head_blocks;
-    if (unit == head_blocks && !write_kv) return;
+    const int token = blockIdx.x, unit = blockIdx.y, head_blocks = gridDim.y - (write_kv ? 1 : 0), heads_per_block = (num_heads + head_blocks - 1) / head_blocks;
     const int position = positions[token];
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(static_cast<float>(position) * inv_freq[i], &sines[i], &cosines[i]);
+    latent_turns(cosines, sines, inv_freq, position, half, factor);
     if (unit < head_blocks) {
         __syncthreads();
         const int head0 = unit * heads_per_block, heads_here = min(num_heads, head0 + heads_per_block) - head0;
@@ -74,25 +142,8 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, con
         }
         return;
     }
-    const T* row = down + static_cast<size_t>(token) * down_stride;
-    float squares = 0.0f;
-    for (int d = threadIdx.x; d < latent; d += blockDim.x) {
-        const float v = to_float(row[d]);
-        squares += v * v;
-    }
-    const float total = block_sum(squares, scratch);   // also orders the writes to cosines[] and sines[]
-    T* dst = latent_row(pages, block_table, layout, token_segment[token], position);
-    if (dst == nullptr) {
-        if (threadIdx.x == 0) report_error(status, kBadPage);
-        return;
-    }
-    const float inv = rsqrtf(total / static_cast<float>(latent) + eps);
-    for (int d = threadIdx.x; d < latent; d += blockDim.x) dst[d] = from_float<T>(to_float(row[d]) * inv * (norm_weight[d] + scale_offset));
-    for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        const float u = to_float(row[latent + i]), v = to_float(row[latent + half + i]);
-        dst[latent + i] = from_float<T>(u * cosines[i] - v * sines[i]);
-        dst[latent + half + i] = from_float<T>(v * cosines[i] + u * sines[i]);
-    }
+    write_latent_row(down + static_cast<size_t>(token) * down_stride, latent_row(pages, block_table, layout, token_segment[token], position), norm_weight, eps,
+                     scale_offset, cosines, sines, scratch, latent, half, status);
 }
 
 constexpr int kLatentThreads = 128, kLatentChunk = 128, kLatentMaxDimsPerThread = 8;   // latent <= 1024
@@ -647,17 +698,35 @@ extern "C" {
 int lb_latent_prepare(const void* q, int q_stride, const void* q_latent, const void* down, int down_stride, void* q_out, void* pages,
                       const float* norm_weight, float eps, float scale_offset, const float* inv_freq, const int* positions, const int* token_segment,
                       const int* block_table, int tokens, int num_heads, int head_dim, int latent, int rope, int page_size, int num_pages, int max_blocks,
-                      int write_kv, int dtype, int* status, cudaStream_t stream) {
+                      int write_kv, int dtype, int* status, cudaStream_t stream, float factor) {
     if (tokens == 0) return 0;
     if (rope < 0 || rope % 2 != 0 || latent < 1 || num_heads < 1) return -2;
     lb::LatentLayout layout{page_size, num_pages, max_blocks, latent, rope};
     const size_t shared = (static_cast<size_t>(rope) + 33) * sizeof(float);
     if (shared > 48 * 1024) return -2;
     LB_DISPATCH_DTYPE(dtype, {
-        lb::latent_prepare_kernel<T><<<dim3(tokens, (q_latent != nullptr ? num_heads : 1) + 1), q_latent != nullptr ? 64 : 128, shared, stream>>>(
+        lb::latent_prepare_kernel<T><<<dim3(tokens, (q_latent != nullptr ? num_heads : 1) + (write_kv ? 1 : 0)), q_latent != nullptr ? 64 : 128, shared, stream>>>(
             static_cast<const T*>(q), q_stride, static_cast<const T*>(q_latent), static_cast<const T*>(down), down_stride, static_cast<T*>(q_out),
             static_cast<T*>(pages), norm_weight, eps, scale_offset, inv_freq, positions, token_segment, block_table, layout, tokens, num_heads, head_dim,
-            write_kv, status);
+            write_kv, status, factor);
+    })
+    return LB_LAUNCH_RESULT();
+}
+
+// q_down and down: column slices of one product, `row_stride` elements a token; down null: no row is written.
+int lb_latent_down(const void* q_down, const void* down, int row_stride, void* q_latent, int q_latent_stride, int q_rank, const float* q_norm_weight, float q_eps,
+                   void* pages, const float* norm_weight, float eps, float scale_offset, const float* inv_freq, float factor, const int* positions,
+                   const int* token_segment, const int* block_table, int tokens, int latent, int rope, int page_size, int num_pages, int max_blocks, int dtype,
+                   int* status, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    if (rope < 0 || rope % 2 != 0 || latent < 1 || q_rank < 1 || q_latent_stride < q_rank) return -2;
+    lb::LatentLayout layout{page_size, num_pages, max_blocks, latent, rope};
+    const size_t shared = (static_cast<size_t>(rope) + 33) * sizeof(float);
+    if (shared > 48 * 1024) return -2;
+    LB_DISPATCH_DTYPE(dtype, {
+        lb::launch_overlapped(lb::latent_down_kernel<T>, dim3(tokens, down != nullptr ? 2 : 1), dim3(tokens <= 64 ? 256 : 128), shared, stream,
+                              static_cast<const T*>(q_down), static_cast<const T*>(down), row_stride, static_cast<T*>(q_latent), q_latent_stride, q_rank, q_norm_weight,
+                              q_eps, static_cast<T*>(pages), norm_weight, eps, scale_offset, inv_freq, factor, positions, token_segment, block_table, layout, status);
     })
     return LB_LAUNCH_RESULT();
 }

@@ -187,6 +187,9 @@ __device__ __forceinline__ float moe_activate(float v, int activation) {
     return v;
 }
 
+// Where a pair's weight multiplies its expert's input (expert(w x) instead of w expert(x)), the two sums are multiplied by it in 32-bit,
+// which is the same since both are linear in the input: `pair_weight` of the kernels below (null: inputs as they are).
+
 // The hidden value of a gated expert from its two 32-bit sums, as a value of T.
 template <typename T>
 __device__ __forceinline__ float moe_hidden(float gate, float up, int activation, float limit) {
@@ -206,7 +209,7 @@ __device__ __forceinline__ float moe_plain_hidden(float up, int activation) {
 template <typename T>
 __global__ void moe_expert_stream_kernel(const T* __restrict__ x, const T* __restrict__ gate, const T* __restrict__ up, const T* __restrict__ down,
                                          const int* __restrict__ chosen, float* __restrict__ out, int top, int width, int ff, int experts,
-                                         int activation, float limit) {
+                                         int activation, float limit, const float* __restrict__ pair_weight) {
     extern __shared__ float shared[];
     float* x_s = shared;           // width
     float* hidden = shared + width;   // ff
@@ -221,6 +224,7 @@ __global__ void moe_expert_stream_kernel(const T* __restrict__ x, const T* __res
     }
     for (int d = threadIdx.x; d < width; d += blockDim.x) x_s[d] = to_float(x[static_cast<size_t>(token) * width + d]);
     __syncthreads();
+    const float factor = pair_weight != nullptr ? pair_weight[pair] : 1.0f;
     const T* up_rows = up + static_cast<size_t>(expert) * ff * width;
     const T* gate_rows = gate != nullptr ? gate + static_cast<size_t>(expert) * ff * width : up_rows;
     for (int f = warp; f < ff; f += warps) {
@@ -231,8 +235,8 @@ __global__ void moe_expert_stream_kernel(const T* __restrict__ x, const T* __res
             if (gate != nullptr) g += x_s[d] * to_float(g_row[d]);
             u += x_s[d] * to_float(u_row[d]);
         }
-        g = warp_sum(g);
-        u = warp_sum(u);
+        g = warp_sum(g) * factor;
+        u = warp_sum(u) * factor;
         if (lane == 0) hidden[f] = gate != nullptr ? moe_hidden<T>(g, u, activation, limit) : moe_plain_hidden<T>(u, activation);
     }
     __syncthreads();
@@ -246,7 +250,7 @@ __global__ void moe_expert_stream_kernel(const T* __restrict__ x, const T* __res
     }
 }
 
-// out[t, :] = T(sum_k weights[t, k] * expert_out[t * top + k, :]), added in the order of k.
+// out[t, :] = T(sum_k weights[t, k] * expert_out[t * top + k, :]), added in the order of k (`weights` null: the plain sum).
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const float* __restrict__ weights, const int* __restrict__ chosen, int experts,
                                    T* __restrict__ out, int top, int width) {
@@ -256,7 +260,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const f
         for (int k = 0; k < top; ++k) {
             const int expert = chosen[static_cast<size_t>(token) * top + k];
             if (expert < 0 || expert >= experts) continue;   // no expert: nothing was computed for the pair
-            sum += weights[static_cast<size_t>(token) * top + k] * expert_out[(static_cast<size_t>(token) * top + k) * width + d];
+            sum += (weights != nullptr ? weights[static_cast<size_t>(token) * top + k] : 1.0f) * expert_out[(static_cast<size_t>(token) * top + k) * width + d];
         }
         out[static_cast<size_t>(token) * width + d] = from_float<T>(sum);
     }
@@ -276,7 +280,7 @@ __global__ void moe_combine_add_kernel(const float* __restrict__ expert_out, con
         for (int k = 0; k < top; ++k) {
             const int expert = chosen[static_cast<size_t>(token) * top + k];
             if (expert < 0 || expert >= experts) continue;
-            sum += weights[static_cast<size_t>(token) * top + k] * expert_out[(static_cast<size_t>(token) * top + k) * width + d];
+            sum += (weights != nullptr ? weights[static_cast<size_t>(token) * top + k] : 1.0f) * expert_out[(static_cast<size_t>(token) * top + k) * width + d];
         }
         if (every != nullptr) sum += gate * to_float(every[static_cast<size_t>(token) * width + d]);
         residual[static_cast<size_t>(token) * width + d] += sum;
@@ -331,7 +335,8 @@ __device__ __forceinline__ void four_dots(const float* __restrict__ x_s, const T
 template <typename T>
 __global__ void __launch_bounds__(32 * kStreamWarps)
 moe_gate_up_stream_kernel(const T* __restrict__ x, const T* __restrict__ gate, const T* __restrict__ up, const int* __restrict__ chosen,
-                          T* __restrict__ hidden, int top, int width, int ff, int experts, int activation, float limit) {
+                          T* __restrict__ hidden, int top, int width, int ff, int experts, int activation, float limit,
+                          const float* __restrict__ pair_weight) {
     extern __shared__ float x_s[];   // width
     const int pair = blockIdx.x, token = pair / top, expert = chosen[pair];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -342,6 +347,7 @@ moe_gate_up_stream_kernel(const T* __restrict__ x, const T* __restrict__ gate, c
     }
     for (int d = threadIdx.x; d < width; d += blockDim.x) x_s[d] = to_float(x[static_cast<size_t>(token) * width + d]);
     __syncthreads();
+    const float factor = pair_weight != nullptr ? pair_weight[pair] : 1.0f;
     const T* up_rows = up + static_cast<size_t>(expert) * ff * width;
     const T* gate_rows = gate != nullptr ? gate + static_cast<size_t>(expert) * ff * width : up_rows;
     for (int f0 = first; f0 < min(ff, first + kStreamRowsPerWarp); f0 += 4) {
@@ -357,8 +363,8 @@ moe_gate_up_stream_kernel(const T* __restrict__ x, const T* __restrict__ gate, c
         if (gate != nullptr) four_dots<T>(x_s, g_rows, width, lane, g);
         four_dots<T>(x_s, u_rows, width, lane, u);
         if (lane < 4 && f0 + lane < ff) {
-            const float gv = lane == 0 ? g[0] : lane == 1 ? g[1] : lane == 2 ? g[2] : g[3];
-            const float uv = lane == 0 ? u[0] : lane == 1 ? u[1] : lane == 2 ? u[2] : u[3];
+            const float gv = (lane == 0 ? g[0] : lane == 1 ? g[1] : lane == 2 ? g[2] : g[3]) * factor;
+            const float uv = (lane == 0 ? u[0] : lane == 1 ? u[1] : lane == 2 ? u[2] : u[3]) * factor;
             hidden[static_cast<size_t>(pair) * ff + f0 + lane] = from_float<T>(gate != nullptr ? moe_hidden<T>(gv, uv, activation, limit) : moe_plain_hidden<T>(uv, activation));
         }
     }
@@ -448,7 +454,7 @@ template <int MODE>
 __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const __nv_bfloat16* __restrict__ a_base, const __nv_bfloat16* __restrict__ b_first, const __nv_bfloat16* __restrict__ b_second,
                    const int* __restrict__ offsets, const int* __restrict__ sorted, __nv_bfloat16* __restrict__ hidden_out, float* __restrict__ pair_out,
-                   int experts, int top, int n_total, int k_total, int activation, float limit) {
+                   int experts, int top, int n_total, int k_total, int activation, float limit, const float* __restrict__ pair_weight) {
     constexpr bool GATED = MODE == 1, UP = MODE != 0;   // UP: rows gathered by token, hidden values out
     __shared__ __align__(16) __nv_bfloat16 a_s[2][kGroupedM][kGroupedPitch];
     __shared__ __align__(16) __nv_bfloat16 b_s[GATED ? 2 : 1][2][kGroupedN][kGroupedPitch];
@@ -538,6 +544,7 @@ moe_grouped_kernel(const __nv_bfloat16* __restrict__ a_base, const __nv_bfloat16
     for (int half = 0; half < 2; ++half) {
         const int row = 16 * warp + g + 8 * half;
         if (row >= rows) continue;
+        const float factor = UP && pair_weight != nullptr ? pair_weight[sorted[first + row]] : 1.0f;
 #pragma unroll
         for (int j = 0; j < kGroupedN / 8; ++j) {
 #pragma unroll
@@ -546,11 +553,11 @@ moe_grouped_kernel(const __nv_bfloat16* __restrict__ a_base, const __nv_bfloat16
                 if (n >= n_total) continue;
                 if constexpr (GATED) {
                     using T = __nv_bfloat16;
-                    const float gate_value = acc[0][j][2 * half + e], up_value = acc[1][j][2 * half + e];
+                    const float gate_value = acc[0][j][2 * half + e] * factor, up_value = acc[1][j][2 * half + e] * factor;
                     hidden_out[static_cast<size_t>(first + row) * n_total + n] = from_float<T>(moe_hidden<T>(gate_value, up_value, activation, limit));
                 } else if constexpr (UP) {
                     using T = __nv_bfloat16;
-                    hidden_out[static_cast<size_t>(first + row) * n_total + n] = from_float<T>(moe_plain_hidden<T>(acc[0][j][2 * half + e], activation));
+                    hidden_out[static_cast<size_t>(first + row) * n_total + n] = from_float<T>(moe_plain_hidden<T>(acc[0][j][2 * half + e] * factor, activation));
                 } else {
                     pair_out[static_cast<size_t>(row_source[row]) * n_total + n] = acc[0][j][2 * half + e];
                 }
@@ -590,7 +597,7 @@ int lb_moe_route(const void* x, const float* router, int* chosen, float* weights
 }
 
 int lb_moe_expert_stream(const void* x, const void* gate, const void* up, const void* down, const int* chosen, float* out, int pairs, int top,
-                         int width, int ff, int experts, int activation, int dtype, cudaStream_t stream, float limit) {
+                         int width, int ff, int experts, int activation, int dtype, cudaStream_t stream, float limit, const float* pair_weight) {
     if (pairs == 0) return 0;
     const size_t shared = (static_cast<size_t>(width) + ff) * sizeof(float);
     if (shared > 200 * 1024) return -2;
@@ -598,7 +605,7 @@ int lb_moe_expert_stream(const void* x, const void* gate, const void* up, const 
         auto kernel = lb::moe_expert_stream_kernel<T>;
         if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
         kernel<<<pairs, 256, shared, stream>>>(static_cast<const T*>(x), static_cast<const T*>(gate), static_cast<const T*>(up), static_cast<const T*>(down),
-                                               chosen, out, top, width, ff, experts, activation, limit);
+                                               chosen, out, top, width, ff, experts, activation, limit, pair_weight);
     })
     return LB_LAUNCH_RESULT();
 }
@@ -625,7 +632,7 @@ int lb_moe_combine_add(const float* expert_out, const float* weights, const int*
 // The two products of the few-token path: `hidden` [pairs, ff] in the activation type, `out` [pairs, width] in 32-bit.
 // Rows of 16-byte multiples only (width and ff multiples of 8 for bfloat16, of 4 for float32): -2 otherwise.
 int lb_moe_expert_stream_wide(const void* x, const void* gate, const void* up, const void* down, const int* chosen, void* hidden, float* out, int pairs,
-                              int top, int width, int ff, int experts, int activation, int dtype, cudaStream_t stream, float limit) {
+                              int top, int width, int ff, int experts, int activation, int dtype, cudaStream_t stream, float limit, const float* pair_weight) {
     if (pairs == 0) return 0;
     const int vector = dtype == lb::kBFloat16 ? 8 : 4;
     if (width % vector != 0 || ff % vector != 0 || width * sizeof(float) > 160 * 1024 || ff * sizeof(float) > 160 * 1024) return -2;
@@ -636,7 +643,8 @@ int lb_moe_expert_stream_wide(const void* x, const void* gate, const void* up, c
         if (width * sizeof(float) > 48 * 1024) cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(width * sizeof(float)));
         if (ff * sizeof(float) > 48 * 1024) cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(ff * sizeof(float)));
         first<<<up_grid, 32 * lb::kStreamWarps, width * sizeof(float), stream>>>(static_cast<const T*>(x), static_cast<const T*>(gate), static_cast<const T*>(up), chosen,
-                                                                                static_cast<T*>(hidden), top, width, ff, experts, activation, limit);
+                                                                                static_cast<T*>(hidden), top, width, ff, experts, activation, limit,
+                                                                                pair_weight);
         second<<<down_grid, 32 * lb::kStreamWarps, ff * sizeof(float), stream>>>(static_cast<const T*>(hidden), static_cast<const T*>(down), chosen, out, width, ff, experts);
     })
     return LB_LAUNCH_RESULT();
@@ -646,7 +654,7 @@ int lb_moe_expert_stream_wide(const void* x, const void* gate, const void* up, c
 // `offsets` [experts + 1] and `sorted` [pairs], then the two grouped products.  `hidden` is [pairs, ff] (rows in sorted
 // order), `out` [pairs, width] in 32-bit (rows in pair order; rows of pairs without an expert are not written).
 int lb_moe_experts_grouped(const void* x, const void* gate, const void* up, const void* down, const int* chosen, int* offsets, int* sorted, void* hidden,
-                           float* out, int pairs, int top, int width, int ff, int experts, int activation, cudaStream_t stream, float limit) {
+                           float* out, int pairs, int top, int width, int ff, int experts, int activation, cudaStream_t stream, float limit, const float* pair_weight) {
     if (pairs == 0) return 0;
     if (width % 8 != 0 || ff % 8 != 0 || experts < 1 || experts > 1024) return -2;
     lb::moe_sort_kernel<<<1, 1024, 2 * experts * sizeof(int), stream>>>(chosen, pairs, experts, offsets, sorted);
@@ -655,13 +663,13 @@ int lb_moe_experts_grouped(const void* x, const void* gate, const void* up, cons
     if (gate != nullptr)
         lb::moe_grouped_kernel<1><<<dim3(tiles, (ff + lb::kGroupedN - 1) / lb::kGroupedN), 128, 0, stream>>>(
             x16, static_cast<const __nv_bfloat16*>(gate), static_cast<const __nv_bfloat16*>(up), offsets, sorted, static_cast<__nv_bfloat16*>(hidden), nullptr, experts,
-            top, ff, width, activation, limit);
+            top, ff, width, activation, limit, pair_weight);
     else
         lb::moe_grouped_kernel<2><<<dim3(tiles, (ff + lb::kGroupedN - 1) / lb::kGroupedN), 128, 0, stream>>>(
             x16, static_cast<const __nv_bfloat16*>(up), nullptr, offsets, sorted, static_cast<__nv_bfloat16*>(hidden), nullptr, experts, top, ff, width, activation,
-            limit);
+            limit, pair_weight);
     lb::moe_grouped_kernel<0><<<dim3(tiles, (width + lb::kGroupedN - 1) / lb::kGroupedN), 128, 0, stream>>>(
-        static_cast<const __nv_bfloat16*>(hidden), static_cast<const __nv_bfloat16*>(down), nullptr, offsets, sorted, nullptr, out, experts, top, width, ff, activation, limit);
+        static_cast<const __nv_bfloat16*>(hidden), static_cast<const __nv_bfloat16*>(down), nullptr, offsets, sorted, nullptr, out, experts, top, width, ff, activation, limit, nullptr);
     return LB_LAUNCH_RESULT();
 }
 

@@ -19,7 +19,7 @@ import torch
 
 from . import native
 
-__all__ = ["BiasedSum", "ExpertSum", "KernelError", "ResidualStreams", "ScaledSum", "SlicedSum", "StreamWrite", "dtype_code", "launch_count", "reset_launch_count"]
+__all__ = ["BiasedSum", "ExpertSum", "KernelError", "ResidualStreams", "ResidualTerm", "TermSum", "ScaledSum", "SlicedSum", "StreamWrite", "dtype_code", "launch_count", "reset_launch_count"]
 
 
 class KernelError(RuntimeError):
@@ -92,11 +92,12 @@ class ScaledSum:
 @dataclass
 class ExpertSum:
     """The weighted sum of a token's routed experts left to its consumer: ``sum_k weights[t, k] * pair_out[t * top + k]`` over the
-    pairs whose expert exists, in the order of ``k`` and in 32-bit (:func:`norm_accumulate` adds them on its way; :meth:`sum`
-    gives the plain tensor in ``dtype``)."""
+    pairs whose expert exists, in the order of ``k`` and in 32-bit (:func:`norm_accumulate` and :func:`residual_terms` add them on their
+    way; :meth:`sum` gives the plain tensor in ``dtype``).  ``weights`` of ``None``: the weights are in the experts' inputs already, the
+    sum is a plain one (:func:`norm_accumulate` and :func:`stream_step` take it as :meth:`sum` only)."""
 
     pair_out: torch.Tensor  # float32 [tokens * top, width]
-    weights: torch.Tensor  # float32 [tokens, top]
+    weights: torch.Tensor | None  # float32 [tokens, top]
     chosen: torch.Tensor  # int32 [tokens, top]
     experts: int
     dtype: torch.dtype
@@ -111,6 +112,38 @@ class ExpertSum:
         code = _lib().lb_moe_combine(_ptr(self.pair_out), _ptr(self.weights), _ptr(self.chosen), c_int(self.experts), _ptr(out), c_int(tokens), c_int(top),
                                      c_int(self.pair_out.shape[1]), c_int(dtype_code(self.dtype)), _stream())
         _done(code, "moe_combine")
+        return out
+
+
+@dataclass
+class ResidualTerm:
+    """``value`` (a tensor, a :class:`SlicedSum` or an :class:`ExpertSum`) times ``gate``, a 32-bit number per token, times ``scale``, a
+    32-bit vector over the columns (each may be left out)."""
+
+    value: "torch.Tensor | SlicedSum | ExpertSum"
+    scale: torch.Tensor | None = None
+    gate: torch.Tensor | None = None
+
+
+@dataclass
+class TermSum:
+    """Up to three :class:`ResidualTerm` on their way into the residual stream: whoever reads the stream next adds them first
+    (:func:`residual_terms`, which computes a norm of the sum besides)."""
+
+    terms: list
+
+    @property
+    def shape(self) -> torch.Size:
+        return self.terms[0].value.shape
+
+    def sum(self) -> torch.Tensor:
+        """The plain tensor, in the terms' type (32-bit arithmetic, one rounding)."""
+        value = self.terms[0].value
+        device = (value.partials if isinstance(value, SlicedSum) else value.pair_out if isinstance(value, ExpertSum) else value).device
+        total = torch.zeros(self.shape, dtype=torch.float32, device=device)
+        residual_terms(total, self)
+        out = torch.empty(self.shape, dtype=value.dtype, device=device)
+        cast_rows(total, out)
         return out
 
 
@@ -305,6 +338,9 @@ def _sum_slices(partials: torch.Tensor, out: torch.Tensor, epilogue: str) -> Non
 def residual_add(x: torch.Tensor, delta: torch.Tensor | SlicedSum) -> None:
     """``x += delta`` on the 32-bit residual stream (a :class:`SlicedSum` is summed and rounded first)."""
     _check(x, "x", torch.float32)
+    if isinstance(delta, TermSum):
+        residual_terms(x, delta)
+        return
     if isinstance(delta, BiasedSum):
         delta = delta.sum()
     if isinstance(delta, SlicedSum):
@@ -350,7 +386,7 @@ def norm_accumulate(residual: torch.Tensor, delta: "torch.Tensor | ScaledSum", w
     terms = list(delta.terms) if isinstance(delta, ScaledSum) else [(delta, 1.0, None)]
     if not 1 <= len(terms) <= 2:
         raise KernelError("norm_accumulate: one or two terms")
-    terms = [(tensor.sum() if index > 0 and isinstance(tensor, ExpertSum) else tensor, scale, bias) for index, (tensor, scale, bias) in enumerate(terms)]
+    terms = [(tensor.sum() if isinstance(tensor, ExpertSum) and (index > 0 or tensor.weights is None) else tensor, scale, bias) for index, (tensor, scale, bias) in enumerate(terms)]
     routed = terms[0][0] if isinstance(terms[0][0], ExpertSum) else None
     if routed is not None:
         # the first term comes as the experts' un-summed outputs: the kernel adds them; a stand-in of the right type and shape for the checks below
@@ -388,6 +424,80 @@ def norm_accumulate(residual: torch.Tensor, delta: "torch.Tensor | ScaledSum", w
                                      _ptr(routed.chosen if routed is not None else None), c_int(routed.chosen.shape[1] if routed is not None else 0),
                                      c_int(routed.experts if routed is not None else 0))
     _done(code, "norm_accumulate")
+
+
+MAX_TERMS = 3
+
+
+class _TermRecord(ctypes.Structure):
+    """The kernel's ``ResidualTerm`` (csrc/residual_terms.cu)."""
+
+    _fields_ = [(name, c_void_p) for name in ("rows", "partials", "pair_out", "pair_weight", "pair_expert", "gate", "scale")] + [
+        ("slice_stride", c_longlong)] + [(name, c_int) for name in ("slices", "top", "experts", "gate_stride")]
+
+
+def residual_terms(x: torch.Tensor, terms: TermSum, weight: torch.Tensor | None = None, eps: float = 0.0, out: torch.Tensor | None = None, *,
+                   rows: torch.Tensor | None = None, num_rows: int | None = None, write_back: bool = True) -> None:
+    """``x += sum_i gate_i * scale_i * value_i`` on the 32-bit residual stream and, with ``out``, the RMS norm of the sum,
+    ``out[r] = h / sqrt(mean(h^2) + eps) * weight`` (32-bit throughout, rounded once), in one kernel.  ``rows`` (its first ``num_rows``
+    entries): only these rows, with ``write_back=False`` (the sum is then only worked out, not stored)."""
+    _check(x, "x", torch.float32)
+    tokens, dim = x.shape
+    if not 1 <= len(terms.terms) <= MAX_TERMS:
+        raise KernelError(f"residual_terms: 1 to {MAX_TERMS} terms, not {len(terms.terms)}")
+    dtype = out.dtype if out is not None else None
+    records = (_TermRecord * len(terms.terms))()
+    for record, term in zip(records, terms.terms):
+        value = term.value
+        if tuple(value.shape) != (tokens, dim):
+            raise KernelError("residual_terms: a term and the residual stream differ in shape")
+        if dtype is None:
+            dtype = value.dtype
+        if value.dtype != dtype:
+            raise KernelError("residual_terms: the terms are of one activation type, the output's")
+        if isinstance(value, SlicedSum):
+            _check(value.partials, "partials", torch.float32)
+            record.partials, record.slices, record.slice_stride = value.partials.data_ptr(), value.partials.shape[0], tokens * dim
+        elif isinstance(value, ExpertSum):
+            _check(value.pair_out, "pair_out", torch.float32)
+            _check(value.chosen, "chosen", torch.int32)
+            if value.pair_out.shape[0] != value.chosen.numel():
+                raise KernelError("residual_terms: the experts' outputs and choices do not fit")
+            if value.weights is not None:
+                _check(value.weights, "weights", torch.float32)
+                if value.weights.shape != value.chosen.shape:
+                    raise KernelError("residual_terms: the experts' weights and choices do not fit")
+                record.pair_weight = value.weights.data_ptr()
+            record.pair_out, record.pair_expert, record.top, record.experts = value.pair_out.data_ptr(), value.chosen.data_ptr(), value.chosen.shape[1], value.experts
+        else:
+            _check(value, "term")
+            record.rows = value.data_ptr()
+        if term.scale is not None:
+            _check(term.scale, "scale", torch.float32)
+            if term.scale.numel() != dim:
+                raise KernelError("residual_terms: a scale must have one element per column")
+            record.scale = term.scale.data_ptr()
+        if term.gate is not None:
+            _check(term.gate, "gate", torch.float32)
+            if term.gate.numel() != tokens:
+                raise KernelError("residual_terms: a gate must have one element per token")
+            record.gate, record.gate_stride = term.gate.data_ptr(), 1
+    out_rows = tokens
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+        out_rows = rows.numel() if num_rows is None else num_rows
+        if out_rows > rows.numel() or write_back:
+            raise KernelError("residual_terms: chosen rows are only read, and num_rows of them must be listed")
+    if out is not None:
+        _check(out, "out")
+        if weight is None:
+            raise KernelError("residual_terms: a norm needs its weight")
+        _check(weight, "weight", torch.float32)
+        if out.shape != (out_rows, dim) or weight.numel() != dim:
+            raise KernelError("residual_terms: out must be [rows, dim] and weight [dim]")
+    code = _lib().lb_residual_terms(_ptr(x), records, c_int(len(terms.terms)), _ptr(weight), _ptr(rows), _ptr(out), c_int(out_rows), c_int(dim), c_float(eps),
+                                    c_int(1 if write_back else 0), c_int(dtype_code(dtype)), _stream())
+    _done(code, "residual_terms")
 
 
 def scale_(x: torch.Tensor, factor: float, softcap: float = 0.0) -> None:
@@ -455,6 +565,8 @@ def stream_step(streams: ResidualStreams, update: StreamWrite | None, read: torc
         if update.mix.shape != (count, count) or update.write.numel() != count:
             raise KernelError("stream_step: mix must be [count, count] and write [count]")
         output = update.output
+        if isinstance(output, ExpertSum) and output.weights is None:
+            output = output.sum()
         if tuple(output.shape) != (tokens, dim):
             raise KernelError("stream_step: the sublayer's output must be [tokens, dim]")
         if isinstance(output, BiasedSum):
@@ -1266,34 +1378,71 @@ def _check_latent_pages(pages: torch.Tensor, block_table: torch.Tensor, latent: 
 
 def latent_prepare(q: torch.Tensor, q_latent: torch.Tensor | None, down: torch.Tensor, q_out: torch.Tensor, pages: torch.Tensor, *, norm_weight: torch.Tensor,
                    eps: float, scale_offset: float, inv_freq: torch.Tensor, positions: torch.Tensor, token_segment: torch.Tensor,
-                   block_table: torch.Tensor, num_heads: int, head_dim: int, latent: int, rope: int, write_kv: bool, status: torch.Tensor) -> None:
+                   block_table: torch.Tensor, num_heads: int, head_dim: int, latent: int, rope: int, write_kv: bool, status: torch.Tensor,
+                   turn_scale: float = 1.0) -> None:
     """Latent attention's step between the projections and the attention.  ``q [tokens, heads * (head_dim + rope)]`` and
     ``down [tokens, latent + rope]`` may be column slices of a wider product (row strides are passed on).  Writes the
     row ``[norm(down[:latent]) * (norm_weight + scale_offset) | rope(down[latent:])]`` into the token's page and the
     queries ``[q_latent[h, t] | rope(q[t, h, head_dim:])]`` into ``q_out [tokens, heads, latent + rope]`` (``q_latent=None``:
-    the latent parts are in ``q_out`` already and stay); the rotation pairs channel ``i`` with ``i + rope / 2``."""
+    the latent parts are in ``q_out`` already and stay); the rotation pairs channel ``i`` with ``i + rope / 2``, sines and cosines times
+    ``turn_scale``.  ``write_kv=False``: no row is written, and ``down`` and the norm may be ``None``."""
     tokens = q_out.shape[0]
-    for name, tensor in (("q", q), ("down", down)):
+    for name, tensor in (("q", q), ("down", down))[: 2 if write_kv else 1]:
         if not tensor.is_cuda or tensor.dim() != 2 or tensor.stride(1) != 1 or tensor.dtype != q_out.dtype or tensor.shape[0] != tokens:
             raise KernelError(f"latent_prepare: {name} must be a [tokens, .] CUDA tensor of q_out's type with unit column stride")
     if q_latent is not None:
         _check(q_latent, "q_latent", q_out.dtype)
     _check(q_out, "q_out")
-    _check(norm_weight, "norm_weight", torch.float32)
+    if write_kv:
+        _check(norm_weight, "norm_weight", torch.float32)
     _check(inv_freq, "inv_freq", torch.float32)
     _check(positions, "positions", torch.int32)
     _check(token_segment, "token_segment", torch.int32)
-    if (q.shape[1] != num_heads * (head_dim + rope) or down.shape[1] != latent + rope or (q_latent is not None and q_latent.shape != (num_heads, tokens, latent))
-            or q_out.shape != (tokens, num_heads, latent + rope) or norm_weight.numel() != latent or inv_freq.numel() != rope // 2 or rope % 2):
+    if (q.shape[1] != num_heads * (head_dim + rope) or (write_kv and (down.shape[1] != latent + rope or norm_weight.numel() != latent))
+            or (q_latent is not None and q_latent.shape != (num_heads, tokens, latent))
+            or q_out.shape != (tokens, num_heads, latent + rope) or inv_freq.numel() != rope // 2 or rope % 2):
         raise KernelError("latent_prepare: the sizes of q, q_latent, down, q_out, the norm's weight and the frequencies do not agree")
     page_size, num_pages, max_blocks = _check_latent_pages(pages, block_table, latent, rope)
     if pages.dtype != q_out.dtype:
         raise KernelError("latent_prepare: cache and activations differ in type")
-    code = _lib().lb_latent_prepare(_ptr(q), c_int(q.stride(0)), _ptr(q_latent), _ptr(down), c_int(down.stride(0)), _ptr(q_out), _ptr(pages), _ptr(norm_weight),
+    code = _lib().lb_latent_prepare(_ptr(q), c_int(q.stride(0)), _ptr(q_latent), _ptr(down if write_kv else None), c_int(down.stride(0) if write_kv else 0), _ptr(q_out), _ptr(pages), _ptr(norm_weight),
                                     c_float(eps), c_float(scale_offset), _ptr(inv_freq), _ptr(positions), _ptr(token_segment), _ptr(block_table), c_int(tokens),
                                     c_int(num_heads), c_int(head_dim), c_int(latent), c_int(rope), c_int(page_size), c_int(num_pages), c_int(max_blocks),
-                                    c_int(1 if write_kv else 0), c_int(dtype_code(q_out.dtype)), _ptr(status), _stream())
+                                    c_int(1 if write_kv else 0), c_int(dtype_code(q_out.dtype)), _ptr(status), _stream(), c_float(turn_scale))
     _done(code, "latent_prepare")
+
+
+def latent_down(q_down: torch.Tensor, down: torch.Tensor | None, q_latent: torch.Tensor, pages: torch.Tensor, *, q_norm_weight: torch.Tensor, q_eps: float,
+                norm_weight: torch.Tensor | None, eps: float, scale_offset: float, inv_freq: torch.Tensor, turn_scale: float, positions: torch.Tensor,
+                token_segment: torch.Tensor, block_table: torch.Tensor, latent: int, rope: int, status: torch.Tensor) -> None:
+    """For latent attention whose queries go through a latent of their own, the step between the down-projections and the queries'
+    up-projection: ``q_latent[t, :q_rank] = norm(q_down[t]) * q_norm_weight`` (zeros in the columns behind, if there are any) and, with ``down``,
+    the token's row in its page (as :func:`latent_prepare` writes it).  ``q_down [tokens, q_rank]`` and ``down [tokens, latent + rope]`` are
+    column slices of one product."""
+    tokens, q_rank = q_down.shape
+    for name, tensor in (("q_down", q_down), ("down", down)):
+        if tensor is not None and (not tensor.is_cuda or tensor.dim() != 2 or tensor.stride(1) != 1 or tensor.dtype != q_latent.dtype or tensor.shape[0] != tokens
+                                   or tensor.stride(0) != q_down.stride(0)):
+            raise KernelError(f"latent_down: {name} must be a column slice of one [tokens, .] CUDA tensor of q_latent's type")
+    _check(q_latent, "q_latent")
+    _check(q_norm_weight, "q_norm_weight", torch.float32)
+    _check(inv_freq, "inv_freq", torch.float32)
+    _check(positions, "positions", torch.int32)
+    _check(token_segment, "token_segment", torch.int32)
+    if q_latent.dim() != 2 or q_latent.shape[0] != tokens or q_latent.shape[1] < q_rank or q_norm_weight.numel() != q_rank or inv_freq.numel() != rope // 2 or rope % 2:
+        raise KernelError("latent_down: the sizes of q_down, q_latent, the norm's weight and the frequencies do not agree")
+    page_size, num_pages, max_blocks = _check_latent_pages(pages, block_table, latent, rope)
+    if pages.dtype != q_latent.dtype:
+        raise KernelError("latent_down: cache and activations differ in type")
+    if down is not None:
+        _check(norm_weight, "norm_weight", torch.float32)
+        if down.shape[1] != latent + rope or norm_weight.numel() != latent:
+            raise KernelError("latent_down: down must be [tokens, latent + rope] with a norm weight of latent elements")
+    code = _lib().lb_latent_down(_ptr(q_down), _ptr(down), c_int(q_down.stride(0)), _ptr(q_latent), c_int(q_latent.shape[1]), c_int(q_rank), _ptr(q_norm_weight),
+                                 c_float(q_eps), _ptr(pages), _ptr(norm_weight), c_float(eps), c_float(scale_offset), _ptr(inv_freq), c_float(turn_scale), _ptr(positions),
+                                 _ptr(token_segment), _ptr(block_table), c_int(tokens), c_int(latent), c_int(rope), c_int(page_size), c_int(num_pages), c_int(max_blocks),
+                                 c_int(dtype_code(q_latent.dtype)), _ptr(status), _stream())
+    _done(code, "latent_down")
 
 
 def _check_sink(sink: torch.Tensor | None, num_heads: int) -> None:
@@ -1453,14 +1602,17 @@ MOE_STREAM_MAX_PAIRS = 32  # up to this many (token, expert) pairs each pair str
 
 
 def moe_experts(x: torch.Tensor, gate: "torch.Tensor | None", up: torch.Tensor, down: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor,
-                activation: str = "silu", path: str | None = None, limit: float = 0.0, combine: bool = True) -> "torch.Tensor | ExpertSum":
+                activation: str = "silu", path: str | None = None, limit: float = 0.0, combine: bool = True,
+                weigh_input: bool = False) -> "torch.Tensor | ExpertSum":
     """``out[t] = sum_k weights[t, k] * down[e] (act(gate[e] x[t]) * (up[e] x[t]))`` with ``e = chosen[t, k]``;
     ``gate`` and ``up`` are ``[experts, ff, width]``, ``down`` ``[experts, width, ff]``.  The weighted sum is
     32-bit, in the order of ``k``; a pair whose expert is no expert counts nothing.  ``path`` forces one of the
     three ways the pairs' products are computed (``"grouped"``, ``"stream"``, ``"plain"``); left out, the sizes
     choose.  ``combine=False`` leaves the weighted sum to the consumer (an :class:`ExpertSum`).  ``gate=None``: experts
-    without a gate, ``down[e] act(up[e] x[t])`` (the activation in 32-bit on the 32-bit sums, rounded once)."""
+    without a gate, ``down[e] act(up[e] x[t])`` (the activation in 32-bit on the 32-bit sums, rounded once).  ``weigh_input``: a weight
+    multiplies its expert's input, not its output, ``sum_k expert_e(weights[t, k] x[t])`` (the 32-bit sums ``gate[e] x`` and ``up[e] x`` are multiplied)."""
     _check(x, "x")
+    input_weight = weights if weigh_input else None
     for name, tensor in (("gate", gate), ("up", up), ("down", down)):
         if tensor is not None:
             _check(tensor, name, x.dtype)
@@ -1490,7 +1642,7 @@ def moe_experts(x: torch.Tensor, gate: "torch.Tensor | None", up: torch.Tensor, 
         order = torch.empty(pairs, dtype=torch.int32, device=x.device)
         hidden = torch.empty(pairs, ff, dtype=x.dtype, device=x.device)
         code = lib.lb_moe_experts_grouped(_ptr(x), _ptr(gate), _ptr(up), _ptr(down), _ptr(chosen), _ptr(offsets), _ptr(order), _ptr(hidden), _ptr(pair_out),
-                                          c_int(pairs), c_int(top), c_int(width), c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), _stream(), c_float(limit))
+                                          c_int(pairs), c_int(top), c_int(width), c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), _stream(), c_float(limit), _ptr(input_weight))
         _done(code, "moe_experts_grouped", 3)
     elif path == "stream":
         # few pairs: each streams its expert's rows, 16 bytes a lane, the rows shared out over many blocks
@@ -1498,18 +1650,19 @@ def moe_experts(x: torch.Tensor, gate: "torch.Tensor | None", up: torch.Tensor, 
             raise KernelError("moe_experts: the streaming kernels take rows of 16-byte multiples")
         hidden = torch.empty(pairs, ff, dtype=x.dtype, device=x.device)
         code = lib.lb_moe_expert_stream_wide(_ptr(x), _ptr(gate), _ptr(up), _ptr(down), _ptr(chosen), _ptr(hidden), _ptr(pair_out), c_int(pairs), c_int(top),
-                                             c_int(width), c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), c_int(dtype_code(x.dtype)), _stream(), c_float(limit))
+                                             c_int(width), c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), c_int(dtype_code(x.dtype)), _stream(), c_float(limit), _ptr(input_weight))
         _done(code, "moe_expert_stream_wide", 2)
     elif path == "plain":
         code = lib.lb_moe_expert_stream(_ptr(x), _ptr(gate), _ptr(up), _ptr(down), _ptr(chosen), _ptr(pair_out), c_int(pairs), c_int(top), c_int(width),
-                                        c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), c_int(dtype_code(x.dtype)), _stream(), c_float(limit))
+                                        c_int(ff), c_int(experts), c_int(_ACTIVATIONS[activation]), c_int(dtype_code(x.dtype)), _stream(), c_float(limit), _ptr(input_weight))
         _done(code, "moe_expert_stream")
     else:
         raise KernelError(f"moe_experts: unknown path {path!r}")
+    output_weight = None if weigh_input else weights
     if not combine:
-        return ExpertSum(pair_out, weights, chosen, experts, x.dtype)   # the consumer adds the pairs' outputs
+        return ExpertSum(pair_out, output_weight, chosen, experts, x.dtype)   # the consumer adds the pairs' outputs
     out = torch.empty(tokens, width, dtype=x.dtype, device=x.device)
-    code = lib.lb_moe_combine(_ptr(pair_out), _ptr(weights), _ptr(chosen), c_int(experts), _ptr(out), c_int(tokens), c_int(top), c_int(width),
+    code = lib.lb_moe_combine(_ptr(pair_out), _ptr(output_weight), _ptr(chosen), c_int(experts), _ptr(out), c_int(tokens), c_int(top), c_int(width),
                               c_int(dtype_code(x.dtype)), _stream())
     _done(code, "moe_combine")
     return out
@@ -1521,10 +1674,11 @@ def moe_combine_add(routed: ExpertSum, residual: torch.Tensor, every: torch.Tens
     a 32-bit number per token (``every_gate`` ``[tokens, 1]`` or ``[tokens]``; left out: 1)."""
     _check(residual, "residual", torch.float32)
     for name, tensor, dtype in (("pair_out", routed.pair_out, torch.float32), ("weights", routed.weights, torch.float32), ("chosen", routed.chosen, torch.int32)):
-        _check(tensor, name, dtype)
+        if tensor is not None:
+            _check(tensor, name, dtype)
     tokens, top = routed.chosen.shape
     width = routed.pair_out.shape[1]
-    if residual.shape != (tokens, width) or routed.pair_out.shape[0] != tokens * top or routed.weights.shape != routed.chosen.shape:
+    if residual.shape != (tokens, width) or routed.pair_out.shape[0] != tokens * top or (routed.weights is not None and routed.weights.shape != routed.chosen.shape):
         raise KernelError("moe_combine_add: the experts' outputs, weights and choices do not fit the residual stream")
     if every is not None:
         _check(every, "every", routed.dtype)
@@ -1563,7 +1717,8 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
                      decay_bias: torch.Tensor | None = None, fixed_decay: torch.Tensor | None = None, tau: float = 1.0, query_scale: float = 1.0,
                      key_scale: float = 1.0, norm_weight: torch.Tensor, norm_eps: float, gate_offset: int | None, gate_activation: str = "silu",
                      segment_start: torch.Tensor, segment_length: torch.Tensor, segment_slot: torch.Tensor, segments: int, status: torch.Tensor,
-                     chunk_plan: dict | None = None, lower: torch.Tensor | None = None, query_silu: bool = False) -> torch.Tensor:
+                     chunk_plan: dict | None = None, lower: torch.Tensor | None = None, query_silu: bool = False, inv_freq: torch.Tensor | None = None,
+                     positions: torch.Tensor | None = None, turn_scale: float = 1.0) -> torch.Tensor:
     """Linear attention ``S_t = diag(a_t) S_(t-1) + k_t v_t^T; o_t = S_t^T q_t`` over the step's portions, from each request's state
     slot and back into it, then the per-head RMS norm of the read-out (times ``norm_weight``) times the gate.
 
@@ -1576,7 +1731,9 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     their decays' products.
 
     ``lower`` (32-bit, ``heads * key_dim``): the decay is ``a = lower + (1 - lower) sigmoid(decay_logits + decay_bias)`` and the key
-    ``1 - a``; ``proj`` then has no key columns (q, v).  ``query_silu``: q is silu of its columns.  ``gate_offset=None``: no gate."""
+    ``1 - a``; ``proj`` then has no key columns (q, v).  ``query_silu``: q is silu of its columns.  ``gate_offset=None``: no gate.
+    ``inv_freq`` (32-bit, one per pair, with ``positions``): channel ``i`` of the first ``2 n`` channels of every head of q and k turns with
+    channel ``i + n`` by ``positions[t] * inv_freq[i]``, sines and cosines times ``turn_scale``, before the scale."""
     _check(proj, "proj")
     _check(matrix_state, "matrix_state", torch.float32)
     _check(norm_weight, "norm_weight", torch.float32)
@@ -1613,6 +1770,11 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
         _check(fixed_decay, "fixed_decay", torch.float32)
         if fixed_decay.numel() != num_heads:
             raise KernelError("linear_attention: fixed_decay must have one element per head")
+    if inv_freq is not None:
+        _check(inv_freq, "inv_freq", torch.float32)
+        if positions is None or lower is not None or query_silu or not 1 <= inv_freq.numel() <= key_dim // 2:
+            raise KernelError("linear_attention: a rotation needs positions and at most key_dim channels, and goes with neither lower bounds nor silu")
+        _check(positions, "positions", torch.int32)
     device = proj.device
     q = torch.empty(tokens, num_heads, key_dim, dtype=torch.float32, device=device)
     k = torch.empty_like(q)
@@ -1622,7 +1784,8 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     code = lib.lb_linear_attention_prepare(_ptr(proj), c_int(proj.shape[1]), _ptr(decay_logits), c_int(decay_logits.stride(0) if decay_logits is not None else 0),
                                            _ptr(decay_bias), _ptr(fixed_decay), c_float(1.0 / tau), c_float(query_scale), c_float(key_scale), _ptr(q), _ptr(k), _ptr(v),
                                            _ptr(decay), c_int(tokens), c_int(num_heads), c_int(key_dim), c_int(value_dim), c_int(dtype_code(proj.dtype)), _stream(),
-                                           _ptr(lower), c_int(1 if query_silu else 0))
+                                           _ptr(lower), c_int(1 if query_silu else 0), _ptr(inv_freq), _ptr(positions if inv_freq is not None else None),
+                                           c_int(2 * inv_freq.numel() if inv_freq is not None else 0), c_float(turn_scale))
     _done(code, "linear_attention_prepare")
     read_out = torch.empty(tokens, num_heads, value_dim, dtype=torch.float32, device=device)
     # the scan of the gated delta rule without its correction (no beta), long portions in chunks where that pays

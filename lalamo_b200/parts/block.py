@@ -21,7 +21,7 @@ import torch
 
 from .base import CacheNeed, CacheView, CompositeNeed, CompositeView, FeedForward, Mixer, Norm, Part, Runtime, StepInputs, TensorDecl, build_part, part_type
 
-__all__ = ["Block", "HyperBlock", "OutputNormBlock", "PreNormBlock", "SandwichNormBlock", "block_tensor_decls", "block_type", "build_block", "register_arrangement"]
+__all__ = ["Block", "HyperBlock", "OutputNormBlock", "ParallelBlock", "PreNormBlock", "SandwichNormBlock", "block_tensor_decls", "block_type", "build_block", "register_arrangement"]
 
 _ARRANGEMENTS: dict[str, type["Block"]] = {}
 
@@ -113,6 +113,46 @@ class PreNormBlock(Block):
         if self.ffn.can_accumulate:
             return self.ffn.forward(normed, step, residual=residual)
         return self.ffn.forward(normed, step)
+
+
+@register_arrangement("parallel")
+class ParallelBlock(Block):
+    """``h = norm(x); x <- x + mixer(h) * mixer_scale + ffn(h) * ffn_scale``: one norm, both sublayers read it, both outputs (times a
+    learned vector each, where there is one) are added at once.  The block leaves its sublayers' outputs un-added and, as far as they
+    come that way, un-summed (``ops.TermSum``): the next block's norm, or the model's last, adds them in 32-bit on its way."""
+
+    roles = ("norm", "mixer", "ffn", "mixer_scale", "ffn_scale")
+    norm: Norm
+    ffn: FeedForward | None
+
+    def __init__(self, spec: Any, tensors: Mapping[tuple[str, str], torch.Tensor], runtime: Runtime) -> None:
+        super().__init__(spec, tensors, runtime)
+        if self.ffn is None and self.ffn_scale is not None:
+            raise ValueError("a parallel block without a feed-forward has no scale for one")
+
+    @staticmethod
+    def _terms(out: Any, scale: Any) -> list:
+        from .. import ops
+
+        vector = scale.scale if scale is not None else None
+        if isinstance(out, ops.TermSum):
+            if vector is None:
+                return out.terms
+            return [ops.ResidualTerm(term.value, vector if term.scale is None else term.scale * vector, term.gate) for term in out.terms]
+        if isinstance(out, (ops.ScaledSum, ops.BiasedSum)):
+            out = out.sum()
+        return [ops.ResidualTerm(out, vector)]
+
+    def forward(self, residual: torch.Tensor, pending: Any, step: StepInputs, cache: CacheView | None) -> Any:
+        from .. import ops
+
+        h = self.norm.residual_forward(residual, pending)
+        mixed = self.mixer.forward(h, step, cache, defer=True) if self.mixer.can_defer else self.mixer.forward(h, step, cache)
+        terms = self._terms(mixed, self.mixer_scale)
+        if self.ffn is not None:
+            out = self.ffn.forward(h, step, defer=True) if self.ffn.can_defer else self.ffn.forward(h, step)
+            terms += self._terms(out, self.ffn_scale)
+        return ops.TermSum(terms)
 
 
 @register_arrangement("output_norm")
@@ -265,7 +305,7 @@ class HyperBlock(Block):
         from .. import ops
 
         out = part.forward(h, step, *cache, defer=True) if part.can_defer else part.forward(h, step, *cache)
-        return out.sum() if isinstance(out, ops.ScaledSum) else out
+        return out.sum() if isinstance(out, (ops.ScaledSum, ops.TermSum)) else out
 
     def forward(self, residual, pending, step: StepInputs, cache: CompositeView):  # type: ignore[override]
         """``residual``: the streams (``ops.ResidualStreams``) without ``pending`` (an ``ops.StreamWrite`` or ``None``)."""

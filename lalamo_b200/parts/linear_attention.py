@@ -7,7 +7,7 @@ RMS-normed per head, multiplied by an activated gate (if there is one) and proje
 One product gives q, k, v and the gate's logits (rows padded to a multiple of 8); the decay's logits come from two small
 products (the bottleneck padded with zeros to a multiple of 32 columns), those of a forget gate from rows of the first.  A kernel lays the recurrence's inputs out in 32-bit
 with the scale on q or k and the decays; the recurrence is the scan the gated delta rule uses, without that rule's correction;
-the read-out kernel is shared with it too.  Per request the mixer holds the matrix state in 32-bit."""
+the read-out kernel is shared with it too.  A rotation of q and k is part of the first of these kernels.  Per request the mixer holds the matrix state in 32-bit."""
 
 from __future__ import annotations
 
@@ -17,8 +17,8 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..config.plan import LinearAttentionSpec
-from .base import CacheNeed, HostSegments, Mixer, Runtime, SlotStateNeed, SlotStateView, StepInputs, TensorDecl, register_part
+from ..config.plan import LinearAttentionSpec, RopeSpec
+from .base import CacheNeed, HostSegments, Mixer, Runtime, SlotStateNeed, SlotStateView, StepInputs, TensorDecl, build_part, register_part
 
 __all__ = ["LinearAttention"]
 
@@ -79,6 +79,13 @@ class LinearAttention(Mixer):
             self.decay_bias = runtime.vector(tensors["decay_bias"])
         self.norm_weight = runtime.vector(tensors["out_norm"] if spec.norm_weight else torch.ones(dv))
         self.out_proj = runtime.matrix(tensors["out_proj"])
+        self.position = None
+        if spec.position is not None:
+            if not isinstance(spec.position, RopeSpec) or spec.position.pairing != "half" or spec.position.rotary_dim > dk:
+                raise ValueError("linear attention rotates up to key_dim channels of q and k, in halves")
+            if spec.decay == "forget" or spec.query_activation != "identity":
+                raise ValueError("a rotation with keys made from the forget gate or an activation on q is not supported")
+            self.position = build_part(spec.position, {}, runtime)
         scale = dk ** -0.5
         self.query_scale = scale if spec.scaled == "query" else 1.0
         self.key_scale = scale if spec.scaled == "key" else 1.0
@@ -160,6 +167,9 @@ class LinearAttention(Mixer):
             segments=step.segments,
             status=status,
             chunk_plan=chunk_plan,
+            inv_freq=self.position.inv_freq if self.position is not None else None,
+            positions=step.positions,
+            turn_scale=self.position.magnitude if self.position is not None else 1.0,
         )
         if residual is not None:
             return ops.linear_accumulate(read_out, self.out_proj, residual, status=status)

@@ -8,10 +8,10 @@ from typing import Mapping
 import torch
 
 from .. import ops
-from ..config.plan import LayerNormSpec, RMSNormSpec
-from .base import Norm, Runtime, TensorDecl, register_part
+from ..config.plan import LayerNormSpec, LayerScaleSpec, RMSNormSpec
+from .base import Norm, Part, Runtime, TensorDecl, register_part
 
-__all__ = ["LayerNorm", "RMSNorm"]
+__all__ = ["LayerNorm", "LayerScale", "RMSNorm"]
 
 
 @register_part(RMSNormSpec)
@@ -37,11 +37,17 @@ class RMSNorm(Norm):
     def residual_forward(
         self,
         residual: torch.Tensor,
-        delta: "torch.Tensor | ops.SlicedSum | None",
+        delta: "torch.Tensor | ops.SlicedSum | ops.TermSum | None",
         rows: torch.Tensor | None = None,
         num_rows: int | None = None,
     ) -> torch.Tensor:
         out = self._out(residual, rows, num_rows)
+        if isinstance(delta, ops.TermSum):
+            if self.spec.exact and self.spec.scale_offset == 0.0:
+                ops.residual_terms(residual, delta, self.scale, self.spec.eps, out, rows=rows, num_rows=out.shape[0], write_back=rows is None)
+                return out
+            ops.residual_add(residual, delta)
+            delta = None
         ops.rmsnorm(
             residual,
             self.scale,
@@ -107,6 +113,22 @@ class LayerNorm(Norm):
         num_rows: int | None = None,
     ) -> torch.Tensor:
         out = self._out(residual, rows, num_rows)
+        if isinstance(delta, ops.TermSum):
+            ops.residual_add(residual, delta)
+            delta = None
         ops.rmsnorm(residual, self.scale, out, self.spec.eps, delta=delta, rows=rows, write_back=delta is not None and rows is None,
                     exact=True, bias=self.bias, centred=True)
         return out
+
+
+@register_part(LayerScaleSpec)
+class LayerScale(Part):
+    """A learned vector that multiplies a sublayer's output element by element, in 32-bit, where it is added to the stream."""
+
+    def __init__(self, spec: LayerScaleSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        super().__init__(spec, tensors, runtime)
+        self.scale = runtime.vector(tensors["scale"])
+
+    @classmethod
+    def tensor_decls(cls, spec: LayerScaleSpec) -> dict[str, TensorDecl]:
+        return {"scale": TensorDecl((spec.dim,), role="vector", init="ones")}

@@ -55,7 +55,10 @@ class Rope(PositionEncoding):
         if spec.rotary_dim % 2 or spec.rotary_dim <= 0:
             raise ValueError(f"rotary_dim must be positive and even, got {spec.rotary_dim}")
         self.magnitude = 1.0
-        if spec.scaling is None:
+        if spec.scaling is None and spec.exact:
+            index = torch.arange(spec.rotary_dim // 2, dtype=torch.float64)
+            inverse = torch.tensor(float(spec.theta), dtype=torch.float64) ** (-2.0 * index / spec.rotary_dim)
+        elif spec.scaling is None:
             channel = torch.arange(0, spec.rotary_dim, 2, dtype=torch.float32)
             inverse = 1.0 / (torch.tensor(spec.theta, dtype=torch.float32) ** (channel / spec.rotary_dim))
         elif isinstance(spec.scaling, LlamaScaling):

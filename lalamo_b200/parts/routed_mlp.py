@@ -69,7 +69,7 @@ class RoutedMLP(FeedForward):
         """The experts' weighted sum; with a shared feed-forward the two terms are handed on un-summed
         (``ops.ScaledSum``), for a consumer that adds them in 32-bit.  With ``residual`` (the 32-bit stream) everything is
         added to it by one kernel, nothing rounded on the way, and ``None`` is returned.  ``defer``: without a shared
-        feed-forward the weighted sum is left to the consumer (``ops.ExpertSum``)."""
+        feed-forward the weighted sum is left to the consumer (``ops.ExpertSum``), with a gated one both are, with the gate (``ops.TermSum``)."""
         spec = self.spec
         routing = ops.moe_route(x, self.router, top=spec.top, group_count=spec.group_count, group_keep=spec.group_keep, score=spec.score,
                                 renormalize=spec.renormalize, bias=self.router_bias, chosen_softmax=spec.chosen_softmax, weight_scale=spec.weight_scale,
@@ -78,10 +78,15 @@ class RoutedMLP(FeedForward):
         shared_gate = routing[2] if spec.shared_gate else None
         # with a shared feed-forward the consumer adds two terms anyway: the experts' weighted sum is left to it as well
         routed = ops.moe_experts(x, self.gate, self.up, self.down, chosen, weights, spec.activation, limit=spec.limit,
-                                 combine=self.shared is None and residual is None and not defer)
+                                 combine=self.shared is None and residual is None and not defer, weigh_input=spec.weigh_input)
         everyone = None
         if self.shared is not None:
-            everyone = self.shared.forward(x, step)
+            if defer and residual is None and shared_gate is not None and self.shared.can_defer:
+                everyone = self.shared.forward(x, step, defer=True)
+                if not isinstance(everyone, ops.BiasedSum):
+                    return ops.TermSum([ops.ResidualTerm(routed), ops.ResidualTerm(everyone, gate=shared_gate)])
+            else:
+                everyone = self.shared.forward(x, step)
             if isinstance(everyone, (ops.SlicedSum, ops.BiasedSum)):
                 everyone = everyone.sum()
         if residual is not None:
