@@ -325,10 +325,11 @@ def plan_flops(plan, tokens: int, wanted_rows: int = 1) -> float:
         if isinstance(spec, LatentAttentionSpec):
             # projections, the queries taken into the latent's space and the sums taken out of it, scores and sums over latent + rope channels
             heads, full = spec.num_heads, spec.latent_dim + spec.rope_dim
-            rows = heads * (spec.head_dim + spec.rope_dim) + full + (heads * spec.value_dim if spec.gated else 0) + heads * spec.value_dim
+            rows = (spec.query_rank or heads * (spec.head_dim + spec.rope_dim)) + (0 if spec.borrows_kv else full) + (heads * spec.value_dim if spec.gated else 0) + heads * spec.value_dim
             window = spec.window or tokens
             pairs = sum(min(position + 1, window) for position in range(tokens))
-            return 2.0 * rows * spec.model_dim * tokens + 2.0 * heads * (spec.head_dim + spec.value_dim) * spec.latent_dim * tokens + 2.0 * heads * (full + spec.latent_dim) * pairs
+            rank = 2.0 * spec.query_rank * heads * (spec.head_dim + spec.rope_dim) * tokens   # queries through a latent of their own
+            return 2.0 * rows * spec.model_dim * tokens + rank + 2.0 * heads * (spec.head_dim + spec.value_dim) * spec.latent_dim * tokens + 2.0 * heads * (full + spec.latent_dim) * pairs
         if isinstance(spec, GatedDeltaSpec):
             inner = spec.num_heads * (spec.key_dim + spec.value_dim)
             rows = 2 * spec.num_groups * spec.key_dim + 2 * spec.num_heads * spec.value_dim + spec.num_heads + spec.decay_rank + spec.gate_rank
@@ -378,7 +379,9 @@ def run_compare(arguments, peaks: dict, peak_source: str, families: tuple[str, .
     `--config zozenex-compare`: the Zozenex shapes beside the Vuvulorn shapes (attention under a window beside a recurrence with a
     matrix state, routed experts) and the Tudulix shapes (every layer routed, a shared expert).
     `--config mozetar-compare`: the Mozetar shapes beside the Zozenex shapes (linear attention, routed experts) and the Vivulorn shapes
-    (attention over all positions, dense feed-forwards without a gate)."""
+    (attention over all positions, dense feed-forwards without a gate).
+    `--config zevetar-compare`: the Zevetar shapes beside the Tudulix shapes (latent attention under a window, a gated shared expert beside
+    the routed ones) and the Zozenex shapes (retention, every layer routed)."""
     import torch
 
     from lalamo_b200.config import config_from_dict
@@ -559,8 +562,8 @@ def main() -> int:
     parser.add_argument("--steps", type=int, default=500)
     parser.add_argument("--warmup", type=int, default=10)
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    parser.add_argument("--compare-sizes", default="350m,1.2b", help="the sizes --config vuvulorn-compare, tudulix-compare, vivulorn-compare, zozenex-compare and mozetar-compare measure")
-    parser.add_argument("--config", default="lfm2-1.2b-decode", choices=["lfm2-1.2b-decode", "lfm2-350m-mixed", "lfm2-700m-long", "vuvulorn-compare", "tudulix-compare", "vivulorn-compare", "zozenex-compare", "mozetar-compare"],
+    parser.add_argument("--compare-sizes", default="350m,1.2b", help="the sizes --config vuvulorn-compare, tudulix-compare, vivulorn-compare, zozenex-compare, mozetar-compare and zevetar-compare measure")
+    parser.add_argument("--config", default="lfm2-1.2b-decode", choices=["lfm2-1.2b-decode", "lfm2-350m-mixed", "lfm2-700m-long", "vuvulorn-compare", "tudulix-compare", "vivulorn-compare", "zozenex-compare", "mozetar-compare", "zevetar-compare"],
                         help="lfm2-1.2b-decode (default): the decode step and its points; lfm2-350m-mixed: 64 requests with prompts of 128 to 2,048 "
                              "tokens and 256 new tokens through the scheduler; lfm2-700m-long: 16,384-token prompts at batch 1 and 8, then 512 decode steps")
     parser.add_argument("--batch", type=int, default=8)
@@ -607,6 +610,8 @@ def main() -> int:
         return run_compare(arguments, peaks, peak_source, families=("zozenex", "vuvulorn", "tudulix"))
     if arguments.config == "mozetar-compare":
         return run_compare(arguments, peaks, peak_source, families=("mozetar", "zozenex", "vivulorn"))
+    if arguments.config == "zevetar-compare":
+        return run_compare(arguments, peaks, peak_source, families=("zevetar", "tudulix", "zozenex"))
     if arguments.requests:
         requests, prompt_length, new_tokens = (int(part) for part in arguments.requests.split(","))
         engine, config = build_engine(max_tokens=requests * (prompt_length + new_tokens + 64), max_requests=max(requests, 2), max_batch_tokens=2048)

@@ -291,6 +291,10 @@ class ZevetarConfig:
                     return [f"{root}.mlp.e{parts[1]}.{parts[2][:-5]}"]
         raise KeyError(f"Zevetar has no tensor {local!r} at {path!r}")
 
+    def unused_names(self) -> set[str]:
+        """A layer without a feed-forward may still carry its scale."""
+        return {f"l{index}.ls2" for index, layer in enumerate(self.layers) if layer.ffn is None}
+
     def to_json_dict(self) -> dict[str, Any]:
         raw = copy.deepcopy(self.raw)
         raw["architecture"] = "Zevetar"

@@ -117,8 +117,9 @@ __device__ __forceinline__ float term_value_one(const ResidualTerm& term, size_t
 //   h = x[src] + sum_i gate_i[src] * scale_i * value_i[src];   if write_back: x[src] = h
 //   out[r] = T(h * rsqrt(mean(h^2) + eps) * weight)            (out null: only the sum)
 // All of it 32-bit.  Launched to start early, as the plain norm is: it waits for the kernel before it first of all.
+constexpr int kTermThreads = 512;   // at most
 template <typename T>
-__global__ void residual_terms_kernel(float* __restrict__ x, const ResidualTerms terms, const float* __restrict__ weight, const int* __restrict__ rows,
+__global__ void __launch_bounds__(kTermThreads) residual_terms_kernel(float* __restrict__ x, const ResidualTerms terms, const float* __restrict__ weight, const int* __restrict__ rows,
                                       T* __restrict__ out, int dim, float eps, int write_back) {
     extern __shared__ __align__(16) float shared[];
     float* row_cache = shared;           // dim floats
@@ -202,7 +203,7 @@ int lb_residual_terms(float* x, const lb::ResidualTerm* terms, int count, const 
     int threads = dim >= 1024 ? 256 : 128;
     if (out_rows <= 64) {
         threads = ((dim + 3) / 4 + 31) / 32 * 32;
-        threads = threads < 128 ? 128 : (threads > 1024 ? 1024 : threads);
+        threads = threads < 128 ? 128 : (threads > lb::kTermThreads ? lb::kTermThreads : threads);
     }
     LB_DISPATCH_DTYPE(dtype, {
         auto kernel = lb::residual_terms_kernel<T>;

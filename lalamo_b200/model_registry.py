@@ -212,6 +212,26 @@ def _mozetar_shape(width: int, layers: int, heads: int, kv_heads: int, linear_he
             "layers": [entry(index) for index in range(layers)]}
 
 
+def _zevetar_shape(width: int, layers: int, heads: int, linear_heads: int, linear_dim: int, linear_vdim: int, ff: int, experts: int, top: int, query_rank: int, rank: int) -> dict[str, Any]:
+    """A Zevetar shape for the random-weights mode: latent attention (heads of 64 + 32 rotated channels, queries through a latent of ``query_rank``,
+    rows of ``rank`` + 32 channels, a window of 2,048) in turn with retention, every second latent layer on the rows of the one before it; the
+    first layer with a dense feed-forward, the others with ``top`` routed experts of ``ff`` columns and a shared one of as many, which together
+    hold what the dense one holds."""
+    latent = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "q_rank": query_rank, "kv_rank": rank, "scale": 96 ** -0.5, "mask": {"size": 2048},
+              "rot": {"dims": 32, "base": 1000000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    retention = {"heads": linear_heads, "dim": linear_dim, "vdim": linear_vdim, "decay": [1.0 - 2.0 ** (-5 - head) for head in range(linear_heads)],
+                 "rot": {"dims": linear_dim, "base": 1000000.0}}
+    dense = {"kind": "dense", "ff": (top + 1) * ff}
+    routed = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff}}
+
+    def entry(index: int) -> dict[str, Any]:
+        mixer = retention if index % 2 else {**latent, "kv_from": index - 2} if index % 4 == 2 else latent
+        return {"type": "retention" if index % 2 else "latent_attention", "mixer": mixer, "mlp": routed if index else dense}
+
+    return {"architecture": "Zevetar", "vocab": 65536, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": float(width) ** 0.5}, "logit_scale": 1.0,
+            "logit_softcap": 30.0, "layers": [entry(index) for index in range(layers)]}
+
+
 # Shapes of the published checkpoints, and Vuvulorn shapes of the same widths and depths, for the random-weights mode
 # (no weights are downloaded).
 PRESETS: dict[str, dict[str, Any]] = {
@@ -232,4 +252,7 @@ PRESETS: dict[str, dict[str, Any]] = {
     # 16 layers; a dense feed-forward's two matrices (and the three of each of a token's four experts together) hold what the three of a gated one of 4,608 (8,192) columns hold
     "mozetar-350m": _mozetar_shape(1024, 16, 16, 4, 8, 64, 128, 6912, 16, 4),
     "mozetar-1.2b": _mozetar_shape(2048, 16, 16, 4, 8, 128, 128, 12288, 16, 4),
+    # 16 layers; a token's feed-forward columns (3 routed experts + the shared one) are those of the Tudulix shapes, the recurrent heads those of the Zozenex shapes
+    "zevetar-350m": _zevetar_shape(1024, 16, 16, 8, 64, 128, 1152, 16, 3, 512, 256),
+    "zevetar-1.2b": _zevetar_shape(2048, 16, 16, 8, 128, 128, 2048, 16, 3, 768, 256),
 }

@@ -101,7 +101,9 @@ def load_weights(
             problems.wrong_dtype.append((name, info.dtype))
             continue
         found[key] = name
-    problems.unexpected = sorted(name for name in checkpoint if name not in used)
+    # tensors of no effect that a checkpoint of the architecture may carry all the same
+    harmless = set(getattr(config, "unused_names", tuple)())
+    problems.unexpected = sorted(name for name in checkpoint if name not in used and name not in harmless)
     if problems:
         raise problems
     return {key: _convert(checkpoint.read(name), checkpoint[name].dtype, decls[key]).reshape(decls[key].shape) for key, name in found.items()}
