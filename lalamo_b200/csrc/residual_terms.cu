@@ -116,7 +116,7 @@ __device__ __forceinline__ float term_value_one(const ResidualTerm& term, size_t
 // One block per output row r; src = rows ? rows[r] : r.
 //   h = x[src] + sum_i gate_i[src] * scale_i * value_i[src];   if write_back: x[src] = h
 //   out[r] = T(h * rsqrt(mean(h^2) + eps) * weight)            (out null: only the sum)
-// All of it 32-bit.  Launched to start early, as the plain norm is: it waits for the kernel before it first of all.
+// All of it 32-bit.  It may be launched to start early, as the plain norm is: it waits for the kernel before it first of all.
 constexpr int kTermThreads = 512;   // at most
 template <typename T>
 __global__ void __launch_bounds__(kTermThreads) residual_terms_kernel(float* __restrict__ x, const ResidualTerms terms, const float* __restrict__ weight, const int* __restrict__ rows,
@@ -182,9 +182,10 @@ __global__ void __launch_bounds__(kTermThreads) residual_terms_kernel(float* __r
 
 extern "C" {
 
-// terms: `count` records on the host (see ResidualTerm); out null: only the sum (weight is not read then).
+// terms: `count` records on the host (see ResidualTerm); out null: only the sum (weight is not read then).  early 0: launched the ordinary
+// way (where the stream has just waited for another stream).
 int lb_residual_terms(float* x, const lb::ResidualTerm* terms, int count, const float* weight, const int* rows, void* out, int out_rows, int dim, float eps,
-                      int write_back, int dtype, cudaStream_t stream) {
+                      int write_back, int dtype, cudaStream_t stream, int early) {
     if (out_rows == 0) return 0;
     if (count < 0 || count > lb::kMaxTerms || dim < 1 || (out != nullptr && weight == nullptr)) return -2;
     lb::ResidualTerms all = {};
@@ -208,7 +209,8 @@ int lb_residual_terms(float* x, const lb::ResidualTerm* terms, int count, const 
     LB_DISPATCH_DTYPE(dtype, {
         auto kernel = lb::residual_terms_kernel<T>;
         if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
-        lb::launch_overlapped(kernel, dim3(out_rows), dim3(threads), shared, stream, x, all, weight, rows, static_cast<T*>(out), dim, eps, write_back);
+        if (!early) kernel<<<out_rows, threads, shared, stream>>>(x, all, weight, rows, static_cast<T*>(out), dim, eps, write_back);
+        else lb::launch_overlapped(kernel, dim3(out_rows), dim3(threads), shared, stream, x, all, weight, rows, static_cast<T*>(out), dim, eps, write_back);
     })
     return LB_LAUNCH_RESULT();
 }

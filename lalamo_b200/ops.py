@@ -131,6 +131,9 @@ class TermSum:
     (:func:`residual_terms`, which computes a norm of the sum besides)."""
 
     terms: list
+    # True: some of them come from another stream, which the current one has been told to wait for; the kernel that adds them is then
+    # launched the ordinary way, behind everything it depends on
+    joined: bool = False
 
     @property
     def shape(self) -> torch.Size:
@@ -496,7 +499,7 @@ def residual_terms(x: torch.Tensor, terms: TermSum, weight: torch.Tensor | None 
         if out.shape != (out_rows, dim) or weight.numel() != dim:
             raise KernelError("residual_terms: out must be [rows, dim] and weight [dim]")
     code = _lib().lb_residual_terms(_ptr(x), records, c_int(len(terms.terms)), _ptr(weight), _ptr(rows), _ptr(out), c_int(out_rows), c_int(dim), c_float(eps),
-                                    c_int(1 if write_back else 0), c_int(dtype_code(dtype)), _stream())
+                                    c_int(1 if write_back else 0), c_int(dtype_code(dtype)), _stream(), c_int(0 if terms.joined else 1))
     _done(code, "residual_terms")
 
 
@@ -2122,7 +2125,7 @@ USE_TCGEN05_ATTENTION = os.environ.get("LALAMO_B200_TCGEN05_ATTENTION", "1") != 
 # stream faster through the TMA pipeline than through the register-direct kernel.
 TCGEN05_MIN_ROWS_FEW_TOKENS = 16384
 _TC_EPILOGUES = {"store": 0, "store_float": 1, "residual_add": 2, "gated": 4}
-_tc_scratch: dict[int, torch.Tensor] = {}
+_tc_scratch: dict[tuple[int, int], torch.Tensor] = {}  # by device and stream: products on two streams may run at the same time
 _tc_retired: list[torch.Tensor] = []  # outgrown scratch buffers, kept: a recorded graph may hold their address
 # Products cut into K slices hand their partial sums to the next norm instead of summing them in a launch of their own
 # (LALAMO_B200_DEFER_SLICE_SUMS=0 sums at once).
@@ -2201,7 +2204,7 @@ def linear_tcgen05(x: torch.Tensor, weight: torch.Tensor, epilogue: str = "store
         scratch = torch.empty(slices, tokens, rows, dtype=torch.float32, device=x.device)
     elif slices > 1:
         needed = slices * tokens * rows
-        index = x.device.index if x.device.index is not None else torch.cuda.current_device()
+        index = (x.device.index if x.device.index is not None else torch.cuda.current_device(), _stream().value or 0)
         if index not in _tc_scratch or _tc_scratch[index].numel() < needed:
             if index in _tc_scratch:
                 _tc_retired.append(_tc_scratch[index])  # recorded graphs may still write there

@@ -71,6 +71,7 @@ class Runtime:
     device: torch.device
     dtype: torch.dtype  # activation / matrix type: torch.bfloat16 or torch.float32
     status: torch.Tensor = field(default=None)  # type: ignore[assignment]  # int32[1], first kernel error
+    _side_stream: "torch.cuda.Stream | None" = None
 
     def __post_init__(self) -> None:
         if self.dtype not in (torch.bfloat16, torch.float32):
@@ -83,6 +84,12 @@ class Runtime:
 
     def vector(self, tensor: torch.Tensor) -> torch.Tensor:
         return tensor.to(device=self.device, dtype=torch.float32).contiguous()
+
+    def side_stream(self) -> "torch.cuda.Stream":
+        """A second stream, for work that may run beside the current stream's."""
+        if self._side_stream is None:
+            self._side_stream = torch.cuda.Stream(self.device)
+        return self._side_stream
 
     def empty(self, *shape: int, dtype: torch.dtype | None = None) -> torch.Tensor:
         return torch.empty(shape, dtype=dtype or self.dtype, device=self.device)
@@ -294,6 +301,10 @@ class Mixer(Part):
     # True if forward() accepts ``defer=True``: it may then return its output un-summed (an ``ops.SlicedSum``, ``ops.BiasedSum`` or
     # ``ops.ExpertSum``) for a consumer that adds it up on its way.
     can_defer = False
+    # True: its kernels may run at the same time as a feed-forward's on another stream.  What must not happen there: a kernel that lets
+    # its successor start early and then waits for tensor memory, while that successor, or the other stream's kernels, hold it.  The products'
+    # kernels cannot get into this (their shared memory admits no more CTAs to a multiprocessor than its tensor memory has room for).
+    can_fork = False
 
     def forward(self, x: torch.Tensor, step: StepInputs, cache: CacheView | None) -> torch.Tensor | None:
         raise NotImplementedError
@@ -302,6 +313,7 @@ class Mixer(Part):
 class FeedForward(Part):
     can_accumulate = False  # as for Mixer
     can_defer = False
+    can_fork = False  # as for Mixer; and its first kernel is launched the ordinary way, behind everything it depends on
 
     def forward(self, x: torch.Tensor, step: StepInputs) -> torch.Tensor | None:
         raise NotImplementedError

@@ -15,6 +15,7 @@ partial sums of its K slices); ``Norm.residual_forward`` and ``ops.residual_add`
 
 from __future__ import annotations
 
+import os
 from typing import Any, Callable, ClassVar, Mapping
 
 import torch
@@ -23,6 +24,8 @@ from .base import CacheNeed, CacheView, CompositeNeed, CompositeView, FeedForwar
 
 __all__ = ["Block", "HyperBlock", "OutputNormBlock", "ParallelBlock", "PreNormBlock", "SandwichNormBlock", "block_tensor_decls", "block_type", "build_block", "register_arrangement"]
 
+# A parallel block's sublayers on two streams (LALAMO_B200_PARALLEL_STREAMS=0: one after the other).
+PARALLEL_STREAMS = os.environ.get("LALAMO_B200_PARALLEL_STREAMS", "1") != "0"
 _ARRANGEMENTS: dict[str, type["Block"]] = {}
 
 
@@ -119,7 +122,11 @@ class PreNormBlock(Block):
 class ParallelBlock(Block):
     """``h = norm(x); x <- x + mixer(h) * mixer_scale + ffn(h) * ffn_scale``: one norm, both sublayers read it, both outputs (times a
     learned vector each, where there is one) are added at once.  The block leaves its sublayers' outputs un-added and, as far as they
-    come that way, un-summed (``ops.TermSum``): the next block's norm, or the model's last, adds them in 32-bit on its way."""
+    come that way, un-summed (``ops.TermSum``): the next block's norm, or the model's last, adds them in 32-bit on its way.
+
+    The sublayers do not depend on each other: where both allow it they run on two streams (in a recorded step, on two branches of the
+    graph), the feed-forward on the second one.  What that stream's work allocates is only ever used again by that stream, behind the point
+    where it waits for the first one's norm, which is behind whatever read it; what it reads is freed after the streams have joined."""
 
     roles = ("norm", "mixer", "ffn", "mixer_scale", "ffn_scale")
     norm: Norm
@@ -147,12 +154,22 @@ class ParallelBlock(Block):
         from .. import ops
 
         h = self.norm.residual_forward(residual, pending)
+        fork = PARALLEL_STREAMS and self.ffn is not None and self.ffn.can_fork and self.mixer.can_fork
+        others: list = []
+        if fork:
+            main, side = torch.cuda.current_stream(), self.runtime.side_stream()
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                others = self._terms(self._run_ffn(h, step), self.ffn_scale)
         mixed = self.mixer.forward(h, step, cache, defer=True) if self.mixer.can_defer else self.mixer.forward(h, step, cache)
-        terms = self._terms(mixed, self.mixer_scale)
-        if self.ffn is not None:
-            out = self.ffn.forward(h, step, defer=True) if self.ffn.can_defer else self.ffn.forward(h, step)
-            terms += self._terms(out, self.ffn_scale)
-        return ops.TermSum(terms)
+        if fork:
+            main.wait_stream(side)
+        elif self.ffn is not None:
+            others = self._terms(self._run_ffn(h, step), self.ffn_scale)
+        return ops.TermSum(self._terms(mixed, self.mixer_scale) + others, joined=fork)
+
+    def _run_ffn(self, h: torch.Tensor, step: StepInputs) -> Any:
+        return self.ffn.forward(h, step, defer=True) if self.ffn.can_defer else self.ffn.forward(h, step)
 
 
 @register_arrangement("output_norm")

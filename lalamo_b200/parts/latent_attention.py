@@ -121,6 +121,7 @@ class LatentAttention(Mixer):
 
     can_accumulate = True
     can_defer = True
+    can_fork = True
 
     def forward(self, x: torch.Tensor, step: StepInputs, cache: PagedKVView, residual: torch.Tensor | None = None,  # type: ignore[override]
                 defer: bool = False) -> "torch.Tensor | ops.SlicedSum | None":

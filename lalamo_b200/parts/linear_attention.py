@@ -130,6 +130,7 @@ class LinearAttention(Mixer):
 
     can_accumulate = True
     can_defer = True
+    can_fork = True
 
     def forward(self, x: torch.Tensor, step: StepInputs, cache: SlotStateView, residual: torch.Tensor | None = None,  # type: ignore[override]
                 defer: bool = False) -> "torch.Tensor | ops.SlicedSum | None":

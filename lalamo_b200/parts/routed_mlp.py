@@ -64,6 +64,7 @@ class RoutedMLP(FeedForward):
 
     can_accumulate = True
     can_defer = True
+    can_fork = True
 
     def forward(self, x: torch.Tensor, step: StepInputs | None = None, residual: torch.Tensor | None = None, defer: bool = False) -> "torch.Tensor | ops.ScaledSum | ops.ExpertSum | None":
         """The experts' weighted sum; with a shared feed-forward the two terms are handed on un-summed

@@ -247,6 +247,24 @@ def test_recorded_steps_in_bfloat16(models, name):
     compare(load_engine(folder, "bfloat16", cuda_graphs=True), config, weights, requests, schedule, "bfloat16")
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "C"])
+def test_sublayers_on_two_streams_change_nothing(models, name, dtype, monkeypatch):
+    """The two sublayers of a block side by side on two streams, recorded and not, against one after the other: the same bits."""
+    from lalamo_b200.parts import block
+
+    folder, _ = models[name]
+    requests = {key: tokens_for(CONFIGS[name], count, 60 + count) for key, count in (("a", 190), ("b", 70), ("c", 45))}
+    schedule = [[("a", 150), ("b", 2), ("c", 1)], [("a", 1), ("b", 40), ("c", 17)]] + [[("a", 1), ("b", 1), ("c", 1)]] * 27 + [[("a", 12), ("b", 1)]]
+    results = []
+    for together in (True, False):
+        monkeypatch.setattr(block, "PARALLEL_STREAMS", together)
+        for graphs in (True, False):
+            results.append(run_schedule(load_engine(folder, dtype, cuda_graphs=graphs), requests, schedule))
+    for other in results[1:]:
+        assert all(np.array_equal(results[0][key], other[key]) for key in requests)
+
+
 # One row that stands out.  The weights are made so that a cached row's score is tens of units above the others if its token is the marker:
 # a position that sees a marker gets the marker's value, one that sees none about the mean of all others.  A marker that is seen one position
 # early or late, or lost (far back, at a page's border, among the first tokens), changes that row's logits by a good part of their spread.
