@@ -184,8 +184,8 @@ __global__ void __launch_bounds__((kScanCols / kScanThreadCols) * SPLIT)
 gdr_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ g, const float* __restrict__ v,
                 const float* __restrict__ beta, float* __restrict__ state, float* __restrict__ out, const int* __restrict__ segment_start,
                 const int* __restrict__ segment_length, const int* __restrict__ segment_slot, int heads, int groups, int dk, int dv,
-                int num_slots, int* status, const int* __restrict__ segment_list, int v_columns) {
-    // segment_list (may be null): the portions this launch runs.  v_columns <= dv: the columns `v` really has (rows of
+                int num_slots, int* status, const int* __restrict__ segment_list, int v_columns, int from_zero) {
+    // from_zero: the state starts at zero (the slot is only written).  segment_list (may be null): the portions this launch runs.  v_columns <= dv: the columns `v` really has (rows of
     // heads x v_columns); the columns past them get zeros as values (they carry a transition matrix, see the chunked path).
     constexpr int R = kScanThreadRows, C = kScanThreadCols;
     static_assert(DKP == R * SPLIT && SPLIT <= 32, "a column's rows lie in one warp");
@@ -258,7 +258,7 @@ gdr_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const 
     for (int i = 0; i < R; ++i) {
         const int row = ((i >> 2) * SPLIT + part) * 4 + (i & 3);
 #pragma unroll
-        for (int c = 0; c < C; ++c) S[c][i] = (row < dk && column + c < dv) ? S_base[static_cast<size_t>(row) * dv + column + c] : 0.0f;
+        for (int c = 0; c < C; ++c) S[c][i] = (row < dk && column + c < dv && !from_zero) ? S_base[static_cast<size_t>(row) * dv + column + c] : 0.0f;
     }
     int stage = 0;
     for (int t0 = 0; t0 < length; t0 += kBatch, stage ^= 1) {
@@ -455,26 +455,34 @@ gdr_chunk_propagate_kernel(const float* __restrict__ chunk_state, float* __restr
     }
 }
 
-// grid (chunks x tiles of 16 tokens, heads): out[t, h, j] = wide[t, h, j] + sum_m wide[t, h, dv + m] * chunk_in[chunk, h, m, j]
-// for the tile's tokens, which share what is read of chunk_in.
+// grid (chunks x tiles of 16 tokens, heads): out[t, h, j] = base[t, h, j] + sum_m turned[t, h, m] * chunk_in[chunk, h, m, j]
+// for the tile's tokens, which share what is read of chunk_in.  `base` (which may be `out`) and `turned` have rows of their own pitch per
+// token and head.  decay (may be null): one number per head; `turned` then counts decay^(i + 1) times at the chunk's token i.
 constexpr int kReadoutTokens = 16;
-__global__ void gdr_chunk_readout_kernel(const float* __restrict__ wide, const float* __restrict__ chunk_in, const int* __restrict__ chunk_start,
-                                         const int* __restrict__ chunk_length, int tiles_per_chunk, float* __restrict__ out, int heads, int dk, int dv) {
+__global__ void gdr_chunk_readout_kernel(const float* base, int base_pitch, const float* __restrict__ turned, int turned_pitch, const float* __restrict__ decay,
+                                         const float* __restrict__ chunk_in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_length,
+                                         int tiles_per_chunk, float* out, int heads, int dk, int dv) {
     extern __shared__ __align__(16) float r_s[];   // dk x 16: the tokens' values of one m side by side (zeros past the tile's end)
     const int chunk = blockIdx.x / tiles_per_chunk, tile = blockIdx.x - chunk * tiles_per_chunk, head = blockIdx.y;
     const int first = kReadoutTokens * tile, count = min(kReadoutTokens, chunk_length[chunk] - first);
     if (count <= 0) return;
     const int token0 = chunk_start[chunk] + first;
+    const float log_decay = decay != nullptr ? log2f(decay[head]) : 0.0f;
     for (int index = threadIdx.x; index < kReadoutTokens * dk; index += blockDim.x) {
         const int tt = index / dk, m = index - tt * dk;
-        r_s[m * kReadoutTokens + tt] = tt < count ? wide[(static_cast<size_t>(token0 + tt) * heads + head) * (dv + dk) + dv + m] : 0.0f;
+        float r = 0.0f;
+        if (tt < count) {
+            r = turned[(static_cast<size_t>(token0 + tt) * heads + head) * turned_pitch + m];
+            if (decay != nullptr) r *= exp2f(log_decay * static_cast<float>(first + tt + 1));
+        }
+        r_s[m * kReadoutTokens + tt] = r;
     }
     __syncthreads();
     const float* S_in = chunk_in + (static_cast<size_t>(chunk) * heads + head) * dk * dv;
     for (int j = threadIdx.x; j < dv; j += blockDim.x) {
         float sums[kReadoutTokens];
 #pragma unroll
-        for (int tt = 0; tt < kReadoutTokens; ++tt) sums[tt] = tt < count ? wide[(static_cast<size_t>(token0 + tt) * heads + head) * (dv + dk) + j] : 0.0f;
+        for (int tt = 0; tt < kReadoutTokens; ++tt) sums[tt] = tt < count ? base[(static_cast<size_t>(token0 + tt) * heads + head) * base_pitch + j] : 0.0f;
 #pragma unroll 4
         for (int m = 0; m < dk; ++m) {   // four loads of S_in on their way at a time
             const float s = S_in[static_cast<size_t>(m) * dv + j];
@@ -494,20 +502,47 @@ __global__ void gdr_chunk_readout_kernel(const float* __restrict__ wide, const f
     }
 }
 
+// One fixed decay a per head, no correction: a chunk of L tokens turns S_in into a^L S_in + S0_L, element by element, so chunks need no
+// further columns.  grid (long portions, heads, pieces of dk * dv), threads over the elements; tables as above, chunk_state [chunks, heads, dk, dv].
+__global__ void retention_chunk_propagate_kernel(const float* __restrict__ chunk_state, float* __restrict__ chunk_in, float* __restrict__ state,
+                                                 const int* __restrict__ long_table, const int* __restrict__ segment_slot, const int* __restrict__ chunk_length,
+                                                 const float* __restrict__ decay, int heads, int elements, int num_slots) {
+    const int portion = long_table[3 * blockIdx.x], first_chunk = long_table[3 * blockIdx.x + 1], chunks = long_table[3 * blockIdx.x + 2];
+    const int head = blockIdx.y, element = blockIdx.z * blockDim.x + threadIdx.x, slot = segment_slot[portion];
+    if (slot < 0 || slot >= num_slots || element >= elements) return;   // (a bad slot is reported by the host's checks and the scan)
+    const float log_decay = log2f(decay[head]);
+    float* mine = state + (static_cast<size_t>(slot) * heads + head) * elements + element;
+    float s = *mine;
+    for (int c0 = 0; c0 < chunks; c0 += 8) {   // eight chunks' loads on their way at a time
+        float end[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (c0 + u < chunks) end[u] = chunk_state[(static_cast<size_t>(first_chunk + c0 + u) * heads + head) * elements + element];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            if (c0 + u < chunks) {
+                chunk_in[(static_cast<size_t>(first_chunk + c0 + u) * heads + head) * elements + element] = s;
+                s = exp2f(log_decay * static_cast<float>(chunk_length[first_chunk + c0 + u])) * s + end[u];
+            }
+        }
+    }
+    *mine = s;
+}
+
 template <int DKP, int SPLIT>
 inline void launch_scan(dim3 grid, cudaStream_t stream, const float* q, const float* k, const float* g, const float* v, const float* beta,
                         float* state, float* out, const int* segment_start, const int* segment_length, const int* segment_slot, int heads,
-                        int groups, int dk, int dv, int num_slots, int* status, const int* segment_list, int v_columns) {
+                        int groups, int dk, int dv, int num_slots, int* status, const int* segment_list, int v_columns, int from_zero) {
     if (beta != nullptr) {
         static OncePerDevice once;
         allow_shared_memory(once, gdr_scan_kernel<DKP, SPLIT, true>, static_cast<int>(ScanShared<DKP>::kBytes));
         gdr_scan_kernel<DKP, SPLIT, true><<<grid, (kScanCols / kScanThreadCols) * SPLIT, ScanShared<DKP>::kBytes, stream>>>(
-            q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+            q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     } else {
         static OncePerDevice once;
         allow_shared_memory(once, gdr_scan_kernel<DKP, SPLIT, false>, static_cast<int>(ScanShared<DKP>::kBytes));
         gdr_scan_kernel<DKP, SPLIT, false><<<grid, (kScanCols / kScanThreadCols) * SPLIT, ScanShared<DKP>::kBytes, stream>>>(
-            q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+            q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     }
 }
 
@@ -549,23 +584,24 @@ int lb_gdr_conv_state(const void* proj, int proj_width, void* conv_state, const 
     return LB_LAUNCH_RESULT();
 }
 
-// segment_list (may be null): the portions to run, `segments` of them.  v_columns: the columns `v` has (0: dv).
+// segment_list (may be null): the portions to run, `segments` of them.  v_columns: the columns `v` has (0: dv).  from_zero: states start at
+// zero and are only written.
 // beta null: the plain linear recurrence (no delta rule).
 int lb_gdr_scan(const float* q, const float* k, const float* g, const float* v, const float* beta, float* state, float* out,
                 const int* segment_start, const int* segment_length, const int* segment_slot, int segments, int heads, int groups, int dk, int dv,
-                int num_slots, int* status, cudaStream_t stream, const int* segment_list, int v_columns) {
+                int num_slots, int* status, cudaStream_t stream, const int* segment_list, int v_columns, int from_zero) {
     if (segments == 0) return 0;
     if (v_columns <= 0) v_columns = dv;
     if (dk < 1 || dk > 256 || dv < 1 || heads % groups != 0 || v_columns > dv) return -2;
     const dim3 grid(segments, heads, (dv + lb::kScanCols - 1) / lb::kScanCols);
     if (dk <= 32)
-        lb::launch_scan<32, 4>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+        lb::launch_scan<32, 4>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     else if (dk <= 64)
-        lb::launch_scan<64, 8>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+        lb::launch_scan<64, 8>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     else if (dk <= 128)
-        lb::launch_scan<128, 16>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+        lb::launch_scan<128, 16>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     else
-        lb::launch_scan<256, 32>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns);
+        lb::launch_scan<256, 32>(grid, stream, q, k, g, v, beta, state, out, segment_start, segment_length, segment_slot, heads, groups, dk, dv, num_slots, status, segment_list, v_columns, from_zero);
     return LB_LAUNCH_RESULT();
 }
 
@@ -594,7 +630,23 @@ int lb_gdr_chunk_finish(const float* chunk_state, float* chunk_in, float* state,
         chunk_state, chunk_in, state, long_table, segment_slot, heads, dk, dv, num_slots, p_in_shared);
     const int tiles_per_chunk = (chunk_tokens + lb::kReadoutTokens - 1) / lb::kReadoutTokens;
     lb::gdr_chunk_readout_kernel<<<dim3(chunks * tiles_per_chunk, heads), 128, static_cast<size_t>(lb::kReadoutTokens) * dk * sizeof(float), stream>>>(
-        wide, chunk_in, chunk_start, chunk_length, tiles_per_chunk, out, heads, dk, dv);
+        wide, dv + dk, wide + dv, dv + dk, nullptr, chunk_in, chunk_start, chunk_length, tiles_per_chunk, out, heads, dk, dv);
+    return LB_LAUNCH_RESULT();
+}
+
+// The same for one fixed decay per head (see retention_chunk_propagate_kernel): `chunk_state` [chunks, heads, dk, dv] is what the scan over the
+// chunk tables left from zero states; `out` [tokens, heads, dv] holds the chunks' own read-outs and gets what came in; q [tokens, heads, dk].
+int lb_retention_chunk_finish(const float* chunk_state, float* chunk_in, float* state, const float* q, const float* decay, float* out, const int* long_table,
+                              int long_portions, const int* segment_slot, const int* chunk_start, const int* chunk_length, int chunks, int chunk_tokens, int heads,
+                              int dk, int dv, int num_slots, cudaStream_t stream) {
+    if (long_portions == 0 || chunks == 0) return 0;
+    if (dk < 1 || dk > 256 || dv < 1 || chunk_tokens < 1) return -2;
+    const int elements = dk * dv;
+    lb::retention_chunk_propagate_kernel<<<dim3(long_portions, heads, (elements + 255) / 256), 256, 0, stream>>>(chunk_state, chunk_in, state, long_table, segment_slot,
+                                                                                                             chunk_length, decay, heads, elements, num_slots);
+    const int tiles_per_chunk = (chunk_tokens + lb::kReadoutTokens - 1) / lb::kReadoutTokens;
+    lb::gdr_chunk_readout_kernel<<<dim3(chunks * tiles_per_chunk, heads), 128, static_cast<size_t>(lb::kReadoutTokens) * dk * sizeof(float), stream>>>(
+        out, dv, q, dk, decay, chunk_in, chunk_start, chunk_length, tiles_per_chunk, out, heads, dk, dv);
     return LB_LAUNCH_RESULT();
 }
 

@@ -1177,6 +1177,8 @@ def short_conv(
 # ---------------------------------------------------------------------- gated delta rule
 GDR_CHUNK_TOKENS = 256  # long portions are scanned in chunks of this many tokens, side by side
 GDR_LONG_PORTION = 768  # portions of at least this many tokens count as long
+RETENTION_CHUNK_TOKENS = 128  # the same where the decay is one fixed number per head: chunks cost less there
+RETENTION_LONG_PORTION = 384
 
 
 def gated_delta_chunks_pay(key_dim: int, value_dim: int) -> bool:
@@ -1316,7 +1318,7 @@ def gated_delta_rule(
         _done(lib.lb_gdr_chunk_init(_ptr(chunk_state), c_int(num_chunks), c_int(num_heads), c_int(key_dim), c_int(value_dim), _stream()), "gdr_chunk_init")
         code = lib.lb_gdr_scan(_ptr(q), _ptr(k), _ptr(decay), _ptr(v), _ptr(beta), _ptr(chunk_state), _ptr(wide), _ptr(chunk_plan["chunk_start"]),
                                _ptr(chunk_plan["chunk_length"]), _ptr(chunk_plan["chunk_slot"]), c_int(num_chunks), c_int(num_heads), c_int(num_groups),
-                               c_int(key_dim), c_int(wide_dim), c_int(num_chunks), _ptr(status), _stream(), _ptr(None), c_int(value_dim))
+                               c_int(key_dim), c_int(wide_dim), c_int(num_chunks), _ptr(status), _stream(), _ptr(None), c_int(value_dim), c_int(0))
         _done(code, "gdr_scan (chunks)")
         code = lib.lb_gdr_chunk_finish(_ptr(chunk_state), _ptr(chunk_in), _ptr(matrix_state), _ptr(wide), _ptr(read_out), _ptr(chunk_plan["long_table"]),
                                        c_int(num_long), _ptr(segment_slot), _ptr(chunk_plan["chunk_start"]), _ptr(chunk_plan["chunk_length"]), c_int(num_chunks),
@@ -1327,7 +1329,7 @@ def gated_delta_rule(
     if num_direct > 0:
         code = lib.lb_gdr_scan(_ptr(q), _ptr(k), _ptr(decay), _ptr(v), _ptr(beta), _ptr(matrix_state), _ptr(read_out), _ptr(segment_start), _ptr(segment_length),
                                _ptr(segment_slot), c_int(num_direct), c_int(num_heads), c_int(num_groups), c_int(key_dim), c_int(value_dim), c_int(num_slots),
-                               _ptr(status), _stream(), _ptr(direct_list), c_int(value_dim))
+                               _ptr(status), _stream(), _ptr(direct_list), c_int(value_dim), c_int(0))
         _done(code, "gdr_scan")
     out = torch.empty(tokens, num_heads * value_dim, dtype=proj.dtype, device=device)
     code = lib.lb_gdr_output(_ptr(read_out), _ptr(low_rank), c_int(low_rank.stride(0)), c_int(gate_offset), _ptr(norm_weight), _ptr(out), c_int(tokens),
@@ -1793,7 +1795,22 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     read_out = torch.empty(tokens, num_heads, value_dim, dtype=torch.float32, device=device)
     # the scan of the gated delta rule without its correction (no beta), long portions in chunks where that pays
     direct_list, num_direct = None, segments
-    if chunk_plan is not None and chunk_plan["num_chunks"] > 0 and gated_delta_chunks_pay(key_dim, value_dim):
+    if chunk_plan is not None and chunk_plan["num_chunks"] > 0 and fixed_decay is not None:
+        # one number per head: what a chunk does to the state it is given needs no further columns
+        num_chunks, num_long = chunk_plan["num_chunks"], chunk_plan["num_long"]
+        chunk_state = torch.empty(num_chunks, num_heads, key_dim, value_dim, dtype=torch.float32, device=device)
+        chunk_in = torch.empty_like(chunk_state)
+        code = lib.lb_gdr_scan(_ptr(q), _ptr(k), _ptr(decay), _ptr(v), _ptr(None), _ptr(chunk_state), _ptr(read_out), _ptr(chunk_plan["chunk_start"]),
+                               _ptr(chunk_plan["chunk_length"]), _ptr(chunk_plan["chunk_slot"]), c_int(num_chunks), c_int(num_heads), c_int(num_heads),
+                               c_int(key_dim), c_int(value_dim), c_int(num_chunks), _ptr(status), _stream(), _ptr(None), c_int(value_dim), c_int(1))
+        _done(code, "linear_attention_scan (chunks)")
+        code = lib.lb_retention_chunk_finish(_ptr(chunk_state), _ptr(chunk_in), _ptr(matrix_state), _ptr(q), _ptr(fixed_decay), _ptr(read_out), _ptr(chunk_plan["long_table"]),
+                                             c_int(num_long), _ptr(segment_slot), _ptr(chunk_plan["chunk_start"]), _ptr(chunk_plan["chunk_length"]), c_int(num_chunks),
+                                             c_int(chunk_plan.get("chunk_tokens", GDR_CHUNK_TOKENS)), c_int(num_heads), c_int(key_dim), c_int(value_dim), c_int(num_slots),
+                                             _stream())
+        _done(code, "retention_chunk_finish", 2)
+        direct_list, num_direct = chunk_plan["direct"], chunk_plan["num_direct"]
+    elif chunk_plan is not None and chunk_plan["num_chunks"] > 0 and gated_delta_chunks_pay(key_dim, value_dim):
         num_chunks, num_long = chunk_plan["num_chunks"], chunk_plan["num_long"]
         wide_dim = value_dim + key_dim
         wide = torch.empty(tokens, num_heads, wide_dim, dtype=torch.float32, device=device)
@@ -1802,7 +1819,7 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
         _done(lib.lb_gdr_chunk_init(_ptr(chunk_state), c_int(num_chunks), c_int(num_heads), c_int(key_dim), c_int(value_dim), _stream()), "gdr_chunk_init")
         code = lib.lb_gdr_scan(_ptr(q), _ptr(k), _ptr(decay), _ptr(v), _ptr(None), _ptr(chunk_state), _ptr(wide), _ptr(chunk_plan["chunk_start"]),
                                _ptr(chunk_plan["chunk_length"]), _ptr(chunk_plan["chunk_slot"]), c_int(num_chunks), c_int(num_heads), c_int(num_heads),
-                               c_int(key_dim), c_int(wide_dim), c_int(num_chunks), _ptr(status), _stream(), _ptr(None), c_int(value_dim))
+                               c_int(key_dim), c_int(wide_dim), c_int(num_chunks), _ptr(status), _stream(), _ptr(None), c_int(value_dim), c_int(0))
         _done(code, "linear_attention_scan (chunks)")
         code = lib.lb_gdr_chunk_finish(_ptr(chunk_state), _ptr(chunk_in), _ptr(matrix_state), _ptr(wide), _ptr(read_out), _ptr(chunk_plan["long_table"]),
                                        c_int(num_long), _ptr(segment_slot), _ptr(chunk_plan["chunk_start"]), _ptr(chunk_plan["chunk_length"]), c_int(num_chunks),
@@ -1813,7 +1830,7 @@ def linear_attention(proj: torch.Tensor, matrix_state: torch.Tensor, *, num_head
     if num_direct > 0:
         code = lib.lb_gdr_scan(_ptr(q), _ptr(k), _ptr(decay), _ptr(v), _ptr(None), _ptr(matrix_state), _ptr(read_out), _ptr(segment_start), _ptr(segment_length),
                                _ptr(segment_slot), c_int(num_direct), c_int(num_heads), c_int(num_heads), c_int(key_dim), c_int(value_dim), c_int(num_slots),
-                               _ptr(status), _stream(), _ptr(direct_list), c_int(value_dim))
+                               _ptr(status), _stream(), _ptr(direct_list), c_int(value_dim), c_int(0))
         _done(code, "linear_attention_scan")
     out = torch.empty(tokens, num_heads * value_dim, dtype=proj.dtype, device=device)
     gated = gate_offset is not None

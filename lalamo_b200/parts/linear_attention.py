@@ -118,15 +118,21 @@ class LinearAttention(Mixer):
         spec = self.spec
         return SlotStateNeed(shape=(spec.num_heads, spec.key_dim, spec.value_dim), dtype=torch.float32)
 
-    # Long portions run in chunks side by side (the plan the gated delta rule's layers make, shared with them): which rows belong
-    # to which chunk depends on the portions' lengths only.
+    # Long portions run in chunks side by side (the plan the gated delta rule's layers make, shared with them; one of shorter chunks where
+    # the decay is one fixed number per head): which rows belong to which chunk depends on the portions' lengths only.
     step_plan_uses_context = False
 
     def step_plan_key(self) -> object:
-        return ("gated_delta", ops.GDR_CHUNK_TOKENS, ops.GDR_LONG_PORTION)
+        return ("gated_delta", *self._chunking())
+
+    def _chunking(self) -> tuple[int, int]:
+        """``(tokens a chunk, tokens from which on a portion is cut into chunks)``."""
+        if self.spec.decay == "fixed":
+            return ops.RETENTION_CHUNK_TOKENS, ops.RETENTION_LONG_PORTION
+        return ops.GDR_CHUNK_TOKENS, ops.GDR_LONG_PORTION
 
     def plan_step(self, segments: HostSegments) -> dict[str, np.ndarray]:
-        return ops.gated_delta_chunk_plan(segments.start, segments.length)
+        return ops.gated_delta_chunk_plan(segments.start, segments.length, *self._chunking())
 
     can_accumulate = True
     can_defer = True
@@ -139,7 +145,8 @@ class LinearAttention(Mixer):
             raise ValueError("a linear-attention layer cannot read another layer's state")
         status = self.runtime.status
         lists, host_lists = step.plan_of(self)
-        chunk_plan = dict(lists, num_chunks=host_lists["chunk_start"].size, num_long=host_lists["long_table"].size // 3, num_direct=host_lists["direct"].size)
+        chunk_plan = dict(lists, num_chunks=host_lists["chunk_start"].size, num_long=host_lists["long_table"].size // 3, num_direct=host_lists["direct"].size,
+                          chunk_tokens=self._chunking()[0])
         proj = ops.linear(x, self.in_proj, status=status)
         logits = proj[:, self.forget_offset :] if self.forget_offset is not None else None
         if self.decay_down is not None:
